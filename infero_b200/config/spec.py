@@ -45,19 +45,25 @@ MOE_NAMES = (("expert", "mlp.e{}"), ("gate", "gate"), ("up", "up"), ("down", "do
              ("shared", "mlp.shared"), ("shared_gate", "mlp.shared.sg"))
 LATENT_ATTENTION_NAMES = (("q", "mix.q"), ("down", "mix.dkv"), ("latent_norm", "mix.dkv.norm"), ("up_k", "mix.uk"),
                           ("up_v", "mix.uv"), ("gate", "mix.g"), ("o", "mix.o"),
-                          ("q_down", "mix.dq"), ("q_norm", "mix.dq.norm"), ("q_up", "mix.uq"))
+                          ("q_down", "mix.dq"), ("q_norm", "mix.dq.norm"), ("q_up", "mix.uq"), ("sink", "mix.sink"))
 RELU2_NAMES = (("up", "mlp.up"), ("down", "mlp.down"))
 MOE_GROUPED_NAMES = (("expert", "mlp.e{}"), ("gate", "gate"), ("up", "up"), ("down", "down"), ("router", "mlp.router"),
                      ("correction", "mlp.correction"), ("shared", "mlp.shared"))
 NORMED_ATTENTION_NAMES = (("q", "mix.q"), ("k", "mix.k"), ("v", "mix.v"), ("o", "mix.o"), ("gate", "mix.g"),
                           ("q_bias", "mix.q.b"), ("k_bias", "mix.k.b"), ("v_bias", "mix.v.b"),
                           ("q_norm", "mix.q.norm"), ("k_norm", "mix.k.norm"), ("o_bias", "mix.o.b"),
-                          ("distance", "mix.rel"), ("head_mix", "mix.talk"))
+                          ("distance", "mix.rel"), ("head_mix", "mix.talk"), ("sink", "mix.sink"))
 DELTA_MEMORY_NAMES = (("q", "mix.q"), ("k", "mix.k"), ("v", "mix.v"), ("q_conv", "mix.q.conv"), ("k_conv", "mix.k.conv"),
                       ("v_conv", "mix.v.conv"), ("step", "mix.b"), ("decay", "mix.a"), ("dt_bias", "mix.dt_bias"),
                       ("a_log", "mix.A_log"), ("gate", "mix.g"), ("out_norm", "mix.norm"), ("o", "mix.o"))
 GATED_MEMORY_NAMES = (("q", "mix.q"), ("k", "mix.k"), ("v", "mix.v"), ("input", "mix.i"), ("input_bias", "mix.i.b"),
                       ("forget", "mix.f"), ("forget_bias", "mix.f.b"), ("gate", "mix.g"), ("out_norm", "mix.norm"), ("o", "mix.o"))
+CHANNEL_DELTA_NAMES = (("q", "mix.q"), ("k", "mix.k"), ("v", "mix.v"), ("q_conv", "mix.q.conv"), ("k_conv", "mix.k.conv"),
+                       ("v_conv", "mix.v.conv"), ("step", "mix.b"), ("decay_down", "mix.a1"), ("decay_up", "mix.a2"),
+                       ("dt_bias", "mix.dt_bias"), ("a_log", "mix.A_log"), ("gate_down", "mix.g1"), ("gate_up", "mix.g2"),
+                       ("out_norm", "mix.norm"), ("o", "mix.o"))
+DECAYED_MEMORY_NAMES = (("q", "mix.q"), ("k", "mix.k"), ("v", "mix.v"), ("gate", "mix.g"), ("decay_down", "mix.a1"),
+                        ("decay_up", "mix.a2"), ("decay_bias", "mix.a2.b"), ("out_norm", "mix.norm"), ("o", "mix.o"))
 RGLRU_NAMES = (("y", "mix.y"), ("y_bias", "mix.y.b"), ("x", "mix.x"), ("x_bias", "mix.x.b"), ("conv", "mix.conv"),
                ("conv_bias", "mix.conv.b"), ("ra", "mix.ra"), ("ra_bias", "mix.ra.b"), ("ri", "mix.ri"),
                ("ri_bias", "mix.ri.b"), ("lam", "mix.lam"), ("o", "mix.o"))
@@ -66,7 +72,8 @@ SSD_NAMES = (("in", "mix.in"), ("conv", "mix.conv"), ("conv_bias", "mix.conv.b")
 MOE_SCORED_NAMES = (("expert", "mlp.e{}"), ("up", "up"), ("down", "down"), ("router", "mlp.router"), ("shared", "mlp.shared"))
 MIXER_NAMES = {"diff_attention": DIFF_ATTENTION_NAMES, "hgrn2": HGRN2_NAMES, "latent_attention": LATENT_ATTENTION_NAMES,
                "normed_attention": NORMED_ATTENTION_NAMES, "rglru": RGLRU_NAMES, "parallel": (), "ssd": SSD_NAMES,
-               "delta_memory": DELTA_MEMORY_NAMES, "gated_memory": GATED_MEMORY_NAMES}
+               "delta_memory": DELTA_MEMORY_NAMES, "gated_memory": GATED_MEMORY_NAMES,
+               "channel_delta_memory": CHANNEL_DELTA_NAMES, "decayed_memory": DECAYED_MEMORY_NAMES}
 FEED_FORWARD_NAMES = {"moe_swiglu": MOE_NAMES, "relu2": RELU2_NAMES, "moe_grouped": MOE_GROUPED_NAMES,
                       "moe_scored": MOE_SCORED_NAMES}
 
@@ -132,7 +139,7 @@ class MixerSpec:
     query), its value Wuv_n c (``value_dim`` wide).  ``position`` turns the ``rot_dim`` parts of queries and keys
     (its ``rotary_dim`` <= ``rot_dim``; ``rot_dim`` 0: no rotated part at all).  ``out_gate``: head n's result is
     multiplied by sigmoid of the n-th row of one more product of the mixer's input.  Causal softmax over all keys,
-    ``scale`` as given.  ``q_latent_dim`` > 0: the queries go through a latent of their own, q = Wuq rms(Wdq h) w.
+    ``scale`` as given.  ``window``: only that many keys up to the query's own.  ``sink_per_head`` as below.  ``q_latent_dim`` > 0: the queries go through a latent of their own, q = Wuq rms(Wdq h) w.
 
     kind "normed_attention": grouped-query attention whose queries and keys are normed.  ``qk_norm_kind``
     "projection": an RMS norm with a weight over the whole query projection (all heads at once) and over the whole key
@@ -149,6 +156,10 @@ class MixerSpec:
     the bucket of the distance n between query and key: n itself below B // 2, then logarithmically wider buckets up to
     the distance ``distance_max``, beyond which all share the last.  ``head_mix``: the heads' softmax weights are mixed by
     a stored matrix [H, H] before they meet the values: head h applies sum_g T[h, g] weights_g to its own kv head's values.
+    ``sink_per_head``: the softmax's denominator has one more term exp(s_h) with s_h a stored number per head, which nothing
+    else touches.  ``softcap`` = c > 0: a scaled score s becomes c tanh(s / c) before any bias.  ``q_temperature`` = (coef,
+    every): a query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) behind its norm and rotation.
+    ``scale_values``: as a branch of a parallel mixer the layer multiplies its cached values by the branch's scale.
     ``gate_per_channel``: ``out_gate`` has a gate for every number of every head's result instead of one per head.
 
     kind "rglru": a gated linear recurrence over ``rec_width`` channels: a gate branch y = gelu_tanh(Wy h + b) and a
@@ -174,6 +185,15 @@ class MixerSpec:
     cap)) with cap = ``gate_cap``; a running maximum m' = max(f + m, i) from 0; S <- exp(f + m - m') S + exp(i - m') k v^T,
     n likewise with k alone; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6).  Every head's o is divided by its root mean
     square; all heads' numbers are multiplied by a weight and by sigmoid(Wg h) and go through the output product.
+
+    kind "channel_delta_memory": the gated delta rule of "delta_memory" with a decay per head and key channel, acting on the rows
+    of S: g = exp(-exp(A_log) softplus(Wa2 (Wa1 h) + dt_bias)) (a product through a narrow middle); the result's gate is
+    sigmoid(Wg2 (Wg1 h)).
+
+    kind "decayed_memory": gated linear attention.  q (times head_dim^(-1/2)), k of ``num_heads`` x ``head_dim``, v of ``num_heads`` x
+    ``value_dim``; decays a = sigmoid(Wa2 (Wa1 h) + b)^(1 / ``decay_tau``) per head and key channel; S <- diag(a) S + k v^T,
+    o = S^T q.  Every head's o is RMS-normed with a weight shared by the heads, multiplied by silu(Wg h) and goes through the
+    output product.
 
     kind "parallel": the mixers of ``branches`` read the same input side by side; the result is the sum of their
     results times ``branch_scales``.  Branch b's tensors carry the leaf names of its own spec.  With ``branch_norms``
@@ -212,6 +232,12 @@ class MixerSpec:
     head_mix: bool = False            # the heads' softmax weights are mixed by a stored matrix
     gate_per_channel: bool = False    # out_gate: one gate per number of a head's result
     gate_cap: float = 0.0             # gated memory: soft bound of the raw gates
+    sink_per_head: bool = False       # a learned sink per head in the softmax's denominator
+    softcap: float = 0.0              # > 0: scaled scores are soft-capped
+    q_temperature: Optional[Tuple[float, float]] = None    # (coef, every): see normed attention
+    scale_values: bool = False        # a branch's scale goes into the cached values
+    low_rank: int = 64                # memories with decays per channel: width of a product's narrow middle where weights are made
+    decay_tau: float = 0.0            # decayed memory: the root taken of its sigmoid
     rec_width: int = 0
     rec_blocks: int = 1
     rec_slope: float = 8.0
@@ -240,7 +266,7 @@ class MixerSpec:
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
-    """kind "swiglu": down(silu(gate(x)) * up(x)) (crates/model/src/lib.rs:7391-7451).
+    """kind "swiglu": down(silu(gate(x)) * up(x)) (crates/model/src/lib.rs:7391-7451); ``bias``: every projection has one.
 
     kind "moe_swiglu": ``experts`` SwiGLU experts of width ``intermediate`` of which every token uses the
     ``top`` with the largest router logits, weighted by the softmax over those logits alone; with
@@ -277,6 +303,7 @@ class FeedForwardSpec:
     route_score: str = "softmax"
     route_renorm: bool = True
     weight_input: bool = False
+    bias: bool = False
     extra: Tuple[Tuple[str, object], ...] = ()
     names: Tuple[Tuple[str, str], ...] = ()          # role -> leaf name (see SWIGLU_NAMES)
     weight_suffix: str = ".weight"
@@ -302,6 +329,7 @@ class BlockSpec:
     kind "sandwich": a norm before and after each sublayer (all of one kind):
     x += post1(mixer(conv(norm1(x)))); x += post2(ffn(norm2(x))); with ``input_conv_name`` the mixer reads
     conv(h) = h + a causal convolution of ``input_conv_taps`` taps per channel over h (no bias), else h itself.
+    kind "postnorm": a norm on each sublayer's result only: x += norm1(mixer(x)); x += norm2(ffn(x)).
     """
     kind: str
     prefix: str
@@ -366,6 +394,8 @@ class ModelSpec:
     bigram: Optional[BigramSpec] = None
     position_table: str = ""          # name of a learned table [max_positions, hidden] added to the embedding ("": none)
     logit_scale: float = 1.0
+    embed_norm: Optional[NormSpec] = None    # an RMS norm of the embedding, what the residual stream starts with
+    embed_norm_name: str = ""
     streams: int = 0                  # > 0: the residual is this many vectors per token, all equal to the embedding at
                                       # the start and added up in front of the final norm (blocks of kind "hyper_prenorm")
 

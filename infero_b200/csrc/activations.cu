@@ -18,12 +18,14 @@ __device__ __forceinline__ float summed(const TI* __restrict__ v, int splits, lo
 
 template <typename TI, typename TO>
 __global__ void glu_act_kernel(const TI* __restrict__ v, int splits, long long split_stride, TO* __restrict__ out, int ff,
-                               size_t total, int kind, float limit, float alpha) {
+                               size_t total, int kind, float limit, float alpha, const float* __restrict__ bias) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     const size_t t = i / ff, j = i % ff;
     const size_t at = t * 2 * ff + 2 * j;
-    out[i] = from_f32<TO>(glu_act(summed(v, splits, split_stride, at), summed(v, splits, split_stride, at + 1), kind, limit, alpha));
+    float g = summed(v, splits, split_stride, at), u = summed(v, splits, split_stride, at + 1);
+    if (bias) g += bias[2 * j], u += bias[2 * j + 1];
+    out[i] = from_f32<TO>(glu_act(g, u, kind, limit, alpha));
 }
 
 template <typename TI, typename TO>
@@ -46,14 +48,15 @@ extern "C" {
         else KERNEL<bf16, bf16><<<blocks, 256, 0, stream>>>((const bf16*)v, splits, split_stride, (bf16*)out, __VA_ARGS__); \
     } while (0)
 
-// v: splits arrays of [n_tokens, 2 * ff], split_stride elements apart; out [n_tokens, ff].
+// v: splits arrays of [n_tokens, 2 * ff], split_stride elements apart; out [n_tokens, ff]; bias (may be null) float32 [2 * ff],
+// added first.
 int infero_glu_act(const void* v, int in_dtype, int splits, long long split_stride, void* out, int out_dtype, int n_tokens,
-                   int ff, int kind, float limit, float alpha, cudaStream_t stream) {
+                   int ff, int kind, float limit, float alpha, const float* bias, cudaStream_t stream) {
     const size_t total = (size_t)n_tokens * ff;
     if (total == 0) return 0;
     INFERO_REQUIRE(splits >= 1 && (kind == GLU_SILU || kind == GLU_CLAMPED), "glu: %d splits, activation %d", splits, kind);
     const unsigned blocks = (unsigned)((total + 255) / 256);
-    DISPATCH(glu_act_kernel, ff, total, kind, limit, alpha);
+    DISPATCH(glu_act_kernel, ff, total, kind, limit, alpha, bias);
     return infero_check_launch("glu_act");
 }
 

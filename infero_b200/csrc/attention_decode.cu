@@ -79,7 +79,7 @@ struct FusedQkv {
 // by zero (what lies in the scratch there may be NaN).
 template <int D>
 __device__ __forceinline__ void merge_if_last(int* counter, float* wbuf, const float* po_base, const float* pml_base,
-                                              int n_splits, int valid, bf16* out_rows, int sink) {
+                                              int n_splits, int valid, bf16* out_rows, int sink, const float* sinks) {
     __shared__ int s_last;
     __syncthreads();                                   // every thread's partial results are written ...
     if (threadIdx.x == 0) {
@@ -130,6 +130,7 @@ __device__ __forceinline__ void merge_if_last(int* counter, float* wbuf, const f
                 }
             }
             if (sink) L += exp2f(-M);                 // the sink's term 2^(0 - M), once for all splits
+            else if (sinks) L += exp2f(sinks[r] - M); // a learned one per head
             const float inv = 1.0f / L;
             uint4 w4;
             w4.x = pack_bf16(a[0] * inv, a[1] * inv);
@@ -167,6 +168,7 @@ __device__ __forceinline__ void merge_if_last(int* counter, float* wbuf, const f
         }
         L = warp_sum(L);
         if (sink) L += exp2f(-M);
+        else if (sinks) L += exp2f(sinks[r] - M);
         if (lane == 0) linv[r] = 1.0f / L;
     }
     __syncthreads();
@@ -275,7 +277,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         if (counters)
             merge_if_last<D>(counters + (size_t)ti * gridDim.y + blockIdx.y, reinterpret_cast<float*>(smem),
                              po - (size_t)split * D, pml - (size_t)split * 2, n_splits, valid,
-                             out + (size_t)t * out_stride + (size_t)row_first * D, sink);
+                             out + (size_t)t * out_stride + (size_t)row_first * D, sink, fq.ex.sinks ? fq.ex.sinks + h0 : nullptr);
         return;
     }
     float2* sc = reinterpret_cast<float2*>(smem + Plan::FUSED_OFFSET);            // [rotary_dim / 2] (sine, cosine)
@@ -487,7 +489,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             }
             __syncwarp();
         }
-        slice16<D, Layout>(qf, kt, vt, 0, kb, lo, pos, lo, pos, scale_log2, m, l, o, lane, bias0, bias1, rel0, rel1, fq.ex.rel_len);
+        slice16<D, Layout>(qf, kt, vt, 0, kb, lo, pos, lo, pos, scale_log2, m, l, o, lane, bias0, bias1, rel0, rel1, fq.ex.rel_len,
+                           fq.ex.cap);
         __syncwarp();
     }
     if (!ok) {
@@ -560,7 +563,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     if (counters)                                      // (its first barrier also ends the reads of red_o above)
         merge_if_last<D>(counters + (size_t)ti * gridDim.y + blockIdx.y, reinterpret_cast<float*>(smem),
                          po - (size_t)split * D, pml - (size_t)split * 2, n_splits, valid,
-                         out + (size_t)t * out_stride + (size_t)row_first * D, sink);
+                         out + (size_t)t * out_stride + (size_t)row_first * D, sink, fq.ex.sinks ? fq.ex.sinks + h0 : nullptr);
     TL_END(TL_ATTN_DECODE);
 }
 
@@ -571,7 +574,7 @@ constexpr int COMBINE_MAX_SPLITS = 256;
 __global__ void __launch_bounds__(128)
 attn_combine_kernel(const float* __restrict__ partial_o, const float* __restrict__ partial_ml,
                     bf16* __restrict__ out, int out_stride, int tok_first, int n_tok, int n_heads,
-                    int n_splits, int head_dim, int sink) {
+                    int n_splits, int head_dim, int sink, const float* __restrict__ sinks, int n_sinks) {
     __shared__ float wsm[4][COMBINE_MAX_SPLITS];
     pdl_launch_dependents();
     pdl_wait();
@@ -593,6 +596,7 @@ attn_combine_kernel(const float* __restrict__ partial_o, const float* __restrict
     float L = 0.f;
     for (int s = 0; s < n_splits; ++s) L += ml[s * 2 + 1] * wgt[s];    // ascending, same in every lane (l is written for every split)
     if (sink) L += exp2f(-M);
+    else if (sinks) L += exp2f(sinks[h % n_sinks] - M);
     const float inv = 1.0f / L;
     bf16* orow = out + (size_t)(tok_first + ti) * out_stride + (size_t)h * head_dim;
     for (int d = lane * 2; d < head_dim; d += 64) {
@@ -680,7 +684,7 @@ int decode_tma(const void* q, int q_stride, const FusedQkv& fq, void* out, int o
     if (rc || counters) return rc;                     // merged by the last CTA of every group
     const int warps = n_tok * per_token;
     launch_pdl(attn_combine_kernel, dim3((warps + 3) / 4), dim3(128), 0, stream, (const float*)po, (const float*)pml,
-               (bf16*)out, out_stride, tok_first, n_tok, per_token, n_splits, head_dim, sink);
+               (bf16*)out, out_stride, tok_first, n_tok, per_token, n_splits, head_dim, sink, fq.ex.sinks, n_heads);
     return infero_check_launch("attn_combine");
 }
 
@@ -721,16 +725,17 @@ int infero_attn_decode_tma_sink(const void* q, int q_stride, void* out, int out_
                       scratch, counters, n_counters, sink, stream);
 }
 
-// The same with what Extras names besides: slopes, a table of biases by distance, the values of every kv head.
+// The same with what Extras names besides: slopes, a table of biases by distance, the values of every kv head, learned
+// sinks (times log2 e), a soft cap of the scaled score (in the score's own units).
 int infero_attn_decode_tma_ex(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
                               const void* v_cache, int num_pages, const int* block_table, int max_blocks,
                               const int* tok_entry, const int* positions, int tok_first, int n_tok, int n_heads,
                               int n_kv, int head_dim, int page_size, int window, float scale, int chunk, int n_splits,
                               void* scratch, int* counters, int n_counters, int sink, const float* slopes, const float* rel,
-                              int rel_len, int cross, cudaStream_t stream) {
+                              int rel_len, int cross, const float* sinks, float softcap, cudaStream_t stream) {
     INFERO_REQUIRE(!rel || rel_len >= 1, "attn_decode_tma: an empty table of distances");
     FusedQkv none = {};
-    none.ex = {slopes, rel, rel_len, cross};
+    none.ex = {slopes, rel, rel_len, cross, sinks, softcap * 1.4426950408889634f};
     return decode_tma(q, q_stride, none, out, out_stride, k_cache, v_cache, num_pages, block_table, max_blocks, tok_entry,
                       positions, tok_first, n_tok, n_heads, n_kv, head_dim, page_size, window, scale, chunk, n_splits,
                       scratch, counters, n_counters, sink, stream);

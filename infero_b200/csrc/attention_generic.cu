@@ -3,7 +3,7 @@
 // For token t of request entry e at position p, head h (kv head h / group):
 //   s_j = (q . K[j]) * scale - slope_h * (p - j)   for lo <= j <= p,  lo = window ? max(0, p - window + 1) : 0
 //   (slope_h: a per-head distance bias, zero where the caller gives no slopes; or a table by distance,
-//   s_j + rel[h][min(p - j, rel_len - 1)])
+//   s_j + rel[h][min(p - j, rel_len - 1)]; with a soft cap the scaled product becomes cap tanh(. / cap) before any bias)
 //   out = sum_j softmax(s)_j V[j]
 // With `cross` head h's weights meet the values of every kv head c, not only its own: out has G * H rows per token, row
 // c * H + h, in 32-bit (what a mixing of the heads' weights needs, see head_mix.cu).
@@ -31,7 +31,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__
                          const int* __restrict__ tok_entry, const int* __restrict__ positions,
                          int n_tokens, int n_heads, int n_kv, int head_dim, int value_dim, int page_size,
                          int window, float scale, int sink, const float* __restrict__ slopes,
-                         const float* __restrict__ rel, int rel_len, int cross) {
+                         const float* __restrict__ rel, int rel_len, int cross, const float* __restrict__ sinks, float softcap) {
     __shared__ float q_s[WARPS][MAX_D];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -52,7 +52,8 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__
 
     // a sink is one more term of the softmax's sum, with score 0 and no value: the running maximum and sum start
     // as if that key had been seen
-    float m = sink ? 0.f : -CUDART_INF_F, l = sink ? 1.f : 0.f;
+    // (with learned sinks its score is the head's own number)
+    float m = sink ? 0.f : sinks ? sinks[h] : -CUDART_INF_F, l = sink || sinks ? 1.f : 0.f;
     float acc[MAX_D / 32];
 #pragma unroll
     for (int i = 0; i < MAX_D / 32; ++i) acc[i] = 0.f;
@@ -69,7 +70,9 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__
                 const T* kr = k_cache + row * head_dim;
                 float d = 0.f;
                 for (int i = 0; i < head_dim; ++i) d = fmaf(q_s[warp][i], to_f32(kr[i]), d);
-                s = d * scale - slope * (float)(pos - j);
+                s = d * scale;
+                if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+                s -= slope * (float)(pos - j);
                 if (rel_h) s += rel_h[min(pos - j, rel_len - 1)];
                 row += (long long)(vh - kvh) * page_size;      // from here on: the row of the values
             }
@@ -111,13 +114,14 @@ extern "C" {
 // the softmax's denominator has one more term exp(0), which carries no value; ``slopes``: float32 [n_heads] or null,
 // head h's score loses slopes[h] times the distance between the query and the key; ``rel``: float32 [n_heads, rel_len] or
 // null, what a score gains at every distance (the last entry also beyond it); ``cross``: every head meets the values of
-// every kv head, out float32 [n_tokens, n_heads * n_kv * value_dim].
+// every kv head, out float32 [n_tokens, n_heads * n_kv * value_dim]; ``sinks``: float32 [n_heads] or null, one more term
+// exp(sinks[h]) of the denominator; ``softcap`` > 0: scaled scores are soft-capped.
 int infero_attention_generic_rel(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
                                  const void* v_cache, int dtype, const int* block_table, int max_blocks,
                                  const int* tok_entry, const int* positions, int n_tokens, int n_heads,
                                  int n_kv, int head_dim, int value_dim, int page_size, int window, float scale,
                                  int sink, const float* slopes, const float* rel, int rel_len, int cross,
-                                 cudaStream_t stream) {
+                                 const float* sinks, float softcap, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     INFERO_REQUIRE(head_dim >= 1 && head_dim <= MAX_D, "attention: head_dim %d outside 1..%d", head_dim, MAX_D);
     INFERO_REQUIRE(value_dim >= 1 && value_dim <= MAX_D, "attention: value width %d outside 1..%d", value_dim, MAX_D);
@@ -128,7 +132,7 @@ int infero_attention_generic_rel(const void* q, int q_stride, void* out, int out
 #define LAUNCH(T, TO)                                                                                                   \
     attention_generic_kernel<T, TO><<<blocks, WARPS * 32, 0, stream>>>((const T*)q, q_stride, (TO*)out, out_stride,     \
         (const T*)k_cache, (const T*)v_cache, block_table, max_blocks, tok_entry, positions, n_tokens, n_heads, n_kv,   \
-        head_dim, value_dim, page_size, window, scale, sink, slopes, rel, rel_len, cross)
+        head_dim, value_dim, page_size, window, scale, sink, slopes, rel, rel_len, cross, sinks, softcap)
     if (dtype == INFERO_F32) LAUNCH(float, float);
     else if (cross) LAUNCH(bf16, float);
     else LAUNCH(bf16, bf16);
@@ -143,7 +147,7 @@ int infero_attention_generic_bias(const void* q, int q_stride, void* out, int ou
                                   int sink, const float* slopes, cudaStream_t stream) {
     return infero_attention_generic_rel(q, q_stride, out, out_stride, k_cache, v_cache, dtype, block_table, max_blocks,
                                         tok_entry, positions, n_tokens, n_heads, n_kv, head_dim, value_dim, page_size,
-                                        window, scale, sink, slopes, nullptr, 0, 0, stream);
+                                        window, scale, sink, slopes, nullptr, 0, 0, nullptr, 0.f, stream);
 }
 
 int infero_attention_generic_ex(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,

@@ -106,7 +106,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
             for (int sl = 0; sl < PF_KEYS / KEYS16; ++sl) {
                 const int kb = key0 + sl * KEYS16;
                 if (kb > warp_hi || kb + KEYS16 <= warp_lo) continue;
-                slice16<D>(qf, kt, kt + TILE, sl * KEYS16, kb, lo0, hi0, lo1, hi1, scale_log2, m, l, o, lane, bias, bias, rel, rel, ex.rel_len);
+                slice16<D>(qf, kt, kt + TILE, sl * KEYS16, kb, lo0, hi0, lo1, hi1, scale_log2, m, l, o, lane, bias, bias, rel, rel, ex.rel_len, ex.cap);
             }
         }
         __syncthreads();
@@ -120,6 +120,9 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
     if (sink) {                       // one more term 2^(0 - m) in the sum, with no value behind it
         l0 += exp2f(-m[0]);
         l1 += exp2f(-m[1]);
+    } else if (ex.sinks) {            // a learned one: 2^(sink - m)
+        l0 += exp2f(ex.sinks[h] - m[0]);
+        l1 += exp2f(ex.sinks[h] - m[1]);
     }
     const float inv0 = 1.0f / l0, inv1 = 1.0f / l1;
     bf16* orow0 = out + (size_t)(tok0 + wrow + g) * out_stride + (size_t)blockIdx.y * D;
@@ -209,7 +212,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
         __syncwarp();
         const bf16* kt = my + (size_t)(i % DEC_STAGES) * 2 * TILE;
         const int kb = k_begin + (warp + i * DEC_WARPS) * KEYS16;
-        slice16<D>(qf, kt, kt + TILE, 0, kb, lo, pos, lo, pos, scale_log2, m, l, o, lane, bias0, bias1, rel0, rel1, ex.rel_len);
+        slice16<D>(qf, kt, kt + TILE, 0, kb, lo, pos, lo, pos, scale_log2, m, l, o, lane, bias0, bias1, rel0, rel1, ex.rel_len, ex.cap);
         __syncwarp();
     }
     cp_async_wait<0>();
@@ -262,7 +265,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
 // ascending order.  One warp per (token, head).
 __global__ void attn_combine_kernel(const float* __restrict__ partial_o, const float* __restrict__ partial_ml,
                                     bf16* __restrict__ out, int out_stride, int tok_first, int n_tok, int n_heads,
-                                    int n_splits, int head_dim, int sink) {
+                                    int n_splits, int head_dim, int sink, const float* __restrict__ sinks, int n_sinks) {
     pdl_launch_dependents();
     pdl_wait();
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
@@ -278,6 +281,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ partial_o, const f
         if (ms != -CUDART_INF_F) L += ml[s * 2 + 1] * exp2f(ms - M);
     }
     if (sink) L += exp2f(-M);          // the sink's term, once for all splits
+    else if (sinks) L += exp2f(sinks[h % n_sinks] - M);
     const float inv = 1.0f / L;
     bf16* orow = out + (size_t)(tok_first + ti) * out_stride + (size_t)h * head_dim;
     for (int d = lane; d < head_dim; d += 32) {
@@ -355,18 +359,20 @@ int infero_attn_mma_supported(int head_dim, int page_size) {
 // of new tokens.  n_tiles = sum over those requests of ceil(q_len / 64).  q / out rows are indexed by the
 // step's token index.
 // ``sink``: the softmax's sum has one more term exp(0) that carries no value.  ``slopes`` (float32 [n_heads] or null):
-// head h's score loses slopes[h] times the distance between the query and the key.  rel, rel_len, cross: see Extras.
+// head h's score loses slopes[h] times the distance between the query and the key.  rel, rel_len, cross, sinks: see
+// Extras; softcap > 0 soft-caps the scaled score (in the score's own units).
 int infero_attn_prefill_ex(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
                            const void* v_cache, const int* block_table, int max_blocks, const int* entry_q_start,
                            const int* entry_q_len, const int* entry_pos0, int n_entries, int first_entry, int n_tiles,
                            int n_heads, int n_kv, int head_dim, int page_size, int window, float scale, int sink,
-                           const float* slopes, const float* rel, int rel_len, int cross, cudaStream_t stream) {
+                           const float* slopes, const float* rel, int rel_len, int cross, const float* sinks, float softcap,
+                           cudaStream_t stream) {
     if (n_tiles == 0) return 0;
     INFERO_REQUIRE(infero_attn_mma_supported(head_dim, page_size), "attn_prefill: head_dim %d / page_size %d not supported", head_dim, page_size);
     INFERO_REQUIRE(n_kv > 0 && n_heads % n_kv == 0 && n_heads * (cross ? n_kv : 1) <= 65535, "attn_prefill: bad head counts %d / %d", n_heads, n_kv);
     INFERO_REQUIRE(q_stride % 2 == 0 && out_stride % 2 == 0, "attn_prefill: odd row strides");
     INFERO_REQUIRE(!rel || rel_len >= 1, "attn_prefill: an empty table of distances");
-    const Extras ex = {slopes, rel, rel_len, cross};
+    const Extras ex = {slopes, rel, rel_len, cross, sinks, softcap * 1.4426950408889634f};
     const float sl2 = scale * 1.4426950408889634f;
 #define CALL(D_) launch_prefill<D_>(q, q_stride, out, out_stride, k_cache, v_cache, block_table, max_blocks, entry_q_start, entry_q_len, entry_pos0, n_entries, first_entry, n_tiles, n_heads, n_kv, page_size, window, sl2, sink, ex, stream)
     DISPATCH_D(head_dim, CALL)
@@ -382,7 +388,7 @@ int infero_attn_prefill_bias(const void* q, int q_stride, void* out, int out_str
                              const float* slopes, cudaStream_t stream) {
     return infero_attn_prefill_ex(q, q_stride, out, out_stride, k_cache, v_cache, block_table, max_blocks, entry_q_start,
                                   entry_q_len, entry_pos0, n_entries, first_entry, n_tiles, n_heads, n_kv, head_dim,
-                                  page_size, window, scale, sink, slopes, nullptr, 0, 0, stream);
+                                  page_size, window, scale, sink, slopes, nullptr, 0, 0, nullptr, 0.f, stream);
 }
 
 int infero_attn_prefill_sink(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
@@ -417,7 +423,8 @@ int infero_attn_decode_ex(const void* q, int q_stride, void* out, int out_stride
                             const void* v_cache, const int* block_table, int max_blocks, const int* tok_entry,
                             const int* positions, int tok_first, int n_tok, int n_heads, int n_kv, int head_dim,
                             int page_size, int window, float scale, int chunk, int n_splits, void* scratch, int sink,
-                            const float* slopes, const float* rel, int rel_len, int cross, cudaStream_t stream) {
+                            const float* slopes, const float* rel, int rel_len, int cross, const float* sinks, float softcap,
+                           cudaStream_t stream) {
     if (n_tok == 0) return 0;
     INFERO_REQUIRE(infero_attn_mma_supported(head_dim, page_size), "attn_decode: head_dim %d / page_size %d not supported", head_dim, page_size);
     INFERO_REQUIRE(n_kv > 0 && n_heads % n_kv == 0, "attn_decode: bad head counts %d / %d", n_heads, n_kv);
@@ -425,7 +432,7 @@ int infero_attn_decode_ex(const void* q, int q_stride, void* out, int out_stride
     INFERO_REQUIRE(n_tok <= 65535, "attn_decode: %d tokens in one call", n_tok);
     INFERO_REQUIRE(q_stride % 2 == 0, "attn_decode: odd row stride");
     INFERO_REQUIRE(!rel || rel_len >= 1, "attn_decode: an empty table of distances");
-    const Extras ex = {slopes, rel, rel_len, cross};
+    const Extras ex = {slopes, rel, rel_len, cross, sinks, softcap * 1.4426950408889634f};
     const int rows = cross ? n_heads * n_kv : n_heads;                // result rows per token
     const float sl2 = scale * 1.4426950408889634f;
     float* po = (float*)scratch;
@@ -448,7 +455,7 @@ int infero_attn_decode_ex(const void* q, int q_stride, void* out, int out_stride
     const int warps = n_tok * rows;
     const int blocks = (warps + 3) / 4;
     attn_combine_kernel<<<blocks, 128, 0, stream>>>(po, pml, (bf16*)out, out_stride, tok_first, n_tok, rows,
-                                                    n_splits, head_dim, sink);
+                                                    n_splits, head_dim, sink, sinks, n_heads);
     return infero_check_launch("attn_combine");
 }
 
@@ -459,7 +466,7 @@ int infero_attn_decode_bias(const void* q, int q_stride, void* out, int out_stri
                             const float* slopes, cudaStream_t stream) {
     return infero_attn_decode_ex(q, q_stride, out, out_stride, k_cache, v_cache, block_table, max_blocks, tok_entry, positions,
                                  tok_first, n_tok, n_heads, n_kv, head_dim, page_size, window, scale, chunk, n_splits, scratch,
-                                 sink, slopes, nullptr, 0, 0, stream);
+                                 sink, slopes, nullptr, 0, 0, nullptr, 0.f, stream);
 }
 
 int infero_attn_decode_sink(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,

@@ -303,6 +303,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         // a table of biases by distance, in the same way
         const float* rel = ex.rel ? ex.rel + (size_t)h * ex.rel_len : nullptr;
         const float inv_scale = 1.0f / scale_log2;
+        // a soft cap: cap tanh(s / cap), again in units of the raw score
+        const float cap = ex.cap * inv_scale, cap_rate = ex.cap > 0.f ? 2.8853900817779268f * scale_log2 / ex.cap : 0.f;
         const uint32_t lane_sel = (uint32_t)((warp & 3) * 32) << 16;
         const uint32_t head_tmem = tmem_base + (uint32_t)t * Plan::HEAD_COLS + lane_sel;
         uint64_t* my_s_full = s_full + t * 2;
@@ -325,6 +327,23 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
             for (int c = 0; c < KTILE / 32; ++c) tmem_ld32_nowait(s_addr + (uint32_t)c * 32u, sv + c * 32);
             tmem_wait_ld();
+            if (ex.cap > 0.f) {
+                // cap (1 - 2 / (1 + e)) with e = e^(2 s / cap), up to 2^25 (from where on a 32-bit tanh is 1); one reciprocal
+                // serves four scores
+                const float two_cap = -2.0f * cap;
+#pragma unroll
+                for (int i = 0; i < KTILE; i += 4) {
+                    float d[4];
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) d[k] = 1.0f + ex2(fminf(__uint_as_float(sv[i + k]) * cap_rate, 25.f));
+                    const float d01 = d[0] * d[1], d23 = d[2] * d[3];
+                    const float r = two_cap * attn::rcp_approx(d01 * d23), r01 = r * d23, r23 = r * d01;
+                    sv[i] = __float_as_uint(fmaf(r01, d[1], cap));
+                    sv[i + 1] = __float_as_uint(fmaf(r01, d[0], cap));
+                    sv[i + 2] = __float_as_uint(fmaf(r23, d[3], cap));
+                    sv[i + 3] = __float_as_uint(fmaf(r23, d[2], cap));
+                }
+            }
             if (bias_k != 0.f) {
                 const float first = (float)(kb - pos_r);                  // key - position of the tile's first key
 #pragma unroll
@@ -417,7 +436,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             // every lane takes part in the TMEM loads (they are warp-wide); only lanes that own a
             // row of the portion store
             // a sink: one more term 2^(0 - m) in the sum, with no value behind it
-            const float inv = 1.0f / (sink ? l + ex2(-m) : l);
+            // (a learned one: 2^(sink - m))
+            const float inv = 1.0f / (sink ? l + ex2(-m) : ex.sinks ? l + ex2(ex.sinks[h] - m) : l);
             const uint32_t o_addr = head_tmem + Plan::O_COL;
             bf16* orow = out + (size_t)(tok0 + row_first + (valid ? r : 0)) * out_stride + (size_t)(ex.cross ? vh * n_heads + h : h) * D;
 #pragma unroll 1
@@ -498,17 +518,18 @@ int infero_attn_prefill_tc_supported(int head_dim, int page_size, int q_stride, 
 // [n_tokens, >= n_heads * head_dim] bf16 with row stride q_stride; the caches are
 // [num_pages, n_kv, page_size, head_dim] bf16, contiguous; all 16-byte aligned.
 // ``sink``: the softmax's sum has one more term exp(0) that carries no value.  ``slopes`` (float32 [n_heads] or null):
-// head h's score loses slopes[h] times the distance between the query and the key.  rel, rel_len, cross: see attn::Extras.
+// head h's score loses slopes[h] times the distance between the query and the key.  rel, rel_len, cross, sinks: see attn::Extras;
+// softcap > 0 soft-caps the scaled score (in the score's own units).
 int infero_attn_prefill_tc_ex(const void* q, int q_stride, int n_tokens, void* out, int out_stride, const void* k_cache,
                                 const void* v_cache, int num_pages, const int* block_table, int max_blocks,
                                 const int* entry_q_start, const int* entry_q_len, const int* entry_pos0, int n_entries,
                                 int first_entry, int n_tiles, int n_heads, int n_kv, int head_dim, int page_size,
                                 int window, float scale, int sink, const float* slopes, const float* rel, int rel_len,
-                              int cross, cudaStream_t stream) {
+                              int cross, const float* sinks, float softcap, cudaStream_t stream) {
     if (n_tiles == 0) return 0;
-    INFERO_REQUIRE((!slopes && !rel) || scale > 0.f, "attn_prefill_tc: a distance bias needs a positive scale");
+    INFERO_REQUIRE((!slopes && !rel && softcap <= 0.f) || scale > 0.f, "attn_prefill_tc: a distance bias or a soft cap needs a positive scale");
     INFERO_REQUIRE(!rel || rel_len >= 1, "attn_prefill_tc: an empty table of distances");
-    const attn::Extras ex = {slopes, rel, rel_len, cross};
+    const attn::Extras ex = {slopes, rel, rel_len, cross, sinks, softcap * 1.4426950408889634f};
     INFERO_REQUIRE(infero_attn_prefill_tc_supported(head_dim, page_size, q_stride, out_stride),
                    "attn_prefill_tc: head_dim %d / page_size %d / strides %d, %d not supported", head_dim, page_size,
                    q_stride, out_stride);
@@ -541,7 +562,7 @@ int infero_attn_prefill_tc_bias(const void* q, int q_stride, int n_tokens, void*
                                 int window, float scale, int sink, const float* slopes, cudaStream_t stream) {
     return infero_attn_prefill_tc_ex(q, q_stride, n_tokens, out, out_stride, k_cache, v_cache, num_pages, block_table,
                                      max_blocks, entry_q_start, entry_q_len, entry_pos0, n_entries, first_entry, n_tiles,
-                                     n_heads, n_kv, head_dim, page_size, window, scale, sink, slopes, nullptr, 0, 0, stream);
+                                     n_heads, n_kv, head_dim, page_size, window, scale, sink, slopes, nullptr, 0, 0, nullptr, 0.f, stream);
 }
 
 int infero_attn_prefill_tc_sink(const void* q, int q_stride, int n_tokens, void* out, int out_stride, const void* k_cache,

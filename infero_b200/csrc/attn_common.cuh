@@ -15,11 +15,31 @@ constexpr int KEYS16 = 16;
 //           times log2(e))
 //   cross   every head's weights meet the values of every kv head: the result has n_kv * n_heads rows per token, row
 //           vh * n_heads + h being head h over kv head vh's values
+//   sinks   float32 [n_heads] or null: the softmax's sum of head h has one more term 2^sinks[h] without a value (a learned
+//           sink, times log2(e)); nothing else touches it
+//   cap     > 0: a score s (scaled) becomes cap tanh(s / cap) before any bias is added; in base-2 units (times log2(e))
 struct Extras {
     const float* slopes;
     const float* rel;
     int rel_len, cross;
+    const float* sinks;
+    float cap;
 };
+
+__device__ __forceinline__ float ex2_approx(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// cap tanh(a / cap) = cap (1 - 2 / (1 + e^(2 a / cap))): off by about cap * 1e-7.  `rate` = 2 log2(e) / cap.
+__device__ __forceinline__ float soft_capped(float a, float cap, float rate) {
+    return fmaf(-2.0f * cap, rcp_approx(1.0f + ex2_approx(fminf(a * rate, 100.f))), cap);
+}
 
 __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
     asm volatile(
@@ -123,14 +143,16 @@ __device__ __forceinline__ void load_q(uint32_t (*qf)[4], const bf16* base, size
 //   (a tile row may hold several keys side by side).
 //   bias0 / bias1: a distance bias of the thread's two rows, in base-2 units per token: the logit of key j loses
 //   bias * (hi - j) (hi is the row's own position wherever a bias is given).
+//   cap > 0: the scaled logit is soft-capped first (Extras).
 //   rel0 / rel1 (null: none): the logit of key j gains rel[min(hi - j, rel_len - 1)], in base-2 units.
 template <int DK, int DV, typename KLayout, typename VLayout>
 __device__ __forceinline__ void slice16_kv(const uint32_t (*qf)[4], const bf16* k_tile, const bf16* v_tile, int row0,
                                            int key_base, int lo0, int hi0, int lo1, int hi1, float scale_log2,
                                            float* m, float* l, float (*o)[4], int lane, int kchunk0 = 0,
                                            float bias0 = 0.f, float bias1 = 0.f, const float* rel0 = nullptr,
-                                           const float* rel1 = nullptr, int rel_len = 0) {
+                                           const float* rel1 = nullptr, int rel_len = 0, float cap = 0.f) {
     const int c = lane & 3;
+    const float cap_rate = cap > 0.f ? 2.8853900817779268f / cap : 0.f;
     float rb[2][4];                                    // (fetched before the products, which they do not depend on)
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
@@ -165,6 +187,10 @@ __device__ __forceinline__ void slice16_kv(const uint32_t (*qf)[4], const bf16* 
         for (int e = 0; e < 2; ++e) {
             const int j = key_base + nt * 8 + c * 2 + e;
             float a = s[nt][e] * scale_log2, b = s[nt][2 + e] * scale_log2;
+            if (cap > 0.f) {
+                a = soft_capped(a, cap, cap_rate);
+                b = soft_capped(b, cap, cap_rate);
+            }
             if (bias0 != 0.f || bias1 != 0.f) {
                 a = fmaf(-bias0, (float)(hi0 - j), a);
                 b = fmaf(-bias1, (float)(hi1 - j), b);
@@ -230,9 +256,10 @@ template <int D, typename Layout = PaddedRows<D>>
 __device__ __forceinline__ void slice16(const uint32_t (*qf)[4], const bf16* k_tile, const bf16* v_tile, int row0,
                                         int key_base, int lo0, int hi0, int lo1, int hi1, float scale_log2,
                                         float* m, float* l, float (*o)[4], int lane, float bias0 = 0.f, float bias1 = 0.f,
-                                        const float* rel0 = nullptr, const float* rel1 = nullptr, int rel_len = 0) {
+                                        const float* rel0 = nullptr, const float* rel1 = nullptr, int rel_len = 0,
+                                        float cap = 0.f) {
     slice16_kv<D, D, Layout, Layout>(qf, k_tile, v_tile, row0, key_base, lo0, hi0, lo1, hi1, scale_log2, m, l, o, lane, 0,
-                                     bias0, bias1, rel0, rel1, rel_len);
+                                     bias0, bias1, rel0, rel1, rel_len, cap);
 }
 
 }  // namespace attn

@@ -279,10 +279,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     continue;
                 }
                 if (EPI == EPI_COL_SWIGLU) {
+                    const float row_bias = bias && ra < RA ? load_any(bias, bias_dtype, ra) : 0.f;
                     // lanes 2j, 2j+1 hold gate_j and up_j of the same tokens: out[rb + i, ra / 2]
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         if (fuse.sumsq_in) v[i] *= col_scale[c0 + i];
+                        v[i] += row_bias;
                         const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);
                         if (!(lane & 1) && ra + 1 < RA && rb + i < RB)
                             out[(size_t)(rb + i) * ldc + (ra >> 1)] = from_f32<OutT>(silu_mul(v[i], other));
@@ -449,6 +451,11 @@ __device__ __forceinline__ void drain_accumulator(uint32_t lane_addr, int ra, in
                 if (EPI == EPI_ROW_SWIGLU) {
                     OutT* dst = out + (size_t)ra * ldc + (rb >> 1);
                     float h[8];
+                    if (bias) {
+#pragma unroll
+                        for (int e = 0; e < 16; ++e)
+                            if (rb + e < RB) v[e] += load_any(bias, bias_dtype, rb + e);
+                    }
 #pragma unroll
                     for (int e = 0; e < 8; ++e)
                         h[e] = act_kind == GLU_SILU ? silu_mul(v[2 * e], v[2 * e + 1])
@@ -1348,8 +1355,9 @@ int infero_gemm_tc(const void* x, const void* w, const void* bias, int bias_dtyp
 // w's rows alternate gate and up.  With few rows this needs the one-split plan (the activation
 // is not linear, so partial sums cannot be combined afterwards): returns 2 when the plan has
 // more than one split, and nothing is launched.
-int infero_gemm_tc_swiglu(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldc,
-                          int sm_count, cudaStream_t stream) {
+// bias (may be null): one number per row of w, added to g and u before the activation.
+int infero_gemm_tc_swiglu_bias(const void* x, const void* w, const void* bias, int bias_dtype, void* out, int M, int N, int K, int ldx,
+                               int ldc, int sm_count, cudaStream_t stream) {
     if (M == 0 || N == 0) return 0;
     INFERO_REQUIRE(infero_gemm_tc_supported(x, w, M, N, K, ldx), "gemm_tc_swiglu: shape M=%d N=%d K=%d ldx=%d not supported", M, N, K, ldx);
     INFERO_REQUIRE(N % 2 == 0 && ldc >= N / 2, "gemm_tc_swiglu: N=%d must be even and ldc=%d at least N/2", N, ldc);
@@ -1364,7 +1372,7 @@ int infero_gemm_tc_swiglu(const void* x, const void* w, void* out, int M, int N,
         CUtensorMap mw, mx;
         if (get_map(w, N, K, K, TILE_A, &mw)) return 1;
         if (get_map(x, M, K, ldx, bn, &mx)) return 1;
-#define GO(BN_, ST_) return launch<BN_, ST_, EPI_COL_SWIGLU, bf16>(mw, mx, out, nullptr, 0, N, M, K, per, 1, ldc, 1, err, stream)
+#define GO(BN_, ST_) return launch<BN_, ST_, EPI_COL_SWIGLU, bf16>(mw, mx, out, bias, bias_dtype, N, M, K, per, 1, ldc, 1, err, stream)
         switch (bn) {
             case 16: GO(16, 6);
             case 32: GO(32, 5);
@@ -1378,10 +1386,15 @@ int infero_gemm_tc_swiglu(const void* x, const void* w, void* out, int M, int N,
     if (get_map(x, M, K, ldx, TILE_A, &mx)) return 1;
     if (get_map(w, N, K, K, 256, &mw)) return 1;
     if (pairs_wanted(M)) {
-        const int r = launch_pair<EPI_ROW_SWIGLU, bf16>(x, w, out, nullptr, 0, M, N, K, ldx, ldc, err, stream);
+        const int r = launch_pair<EPI_ROW_SWIGLU, bf16>(x, w, out, bias, bias_dtype, M, N, K, ldx, ldc, err, stream);
         if (r >= 0) return r;
     }
-    return launch_persistent<EPI_ROW_SWIGLU, bf16>(x, w, out, nullptr, 0, M, N, K, ldx, ldc, sm_count, err, stream);
+    return launch_persistent<EPI_ROW_SWIGLU, bf16>(x, w, out, bias, bias_dtype, M, N, K, ldx, ldc, sm_count, err, stream);
+}
+
+int infero_gemm_tc_swiglu(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldc,
+                          int sm_count, cudaStream_t stream) {
+    return infero_gemm_tc_swiglu_bias(x, w, nullptr, 0, out, M, N, K, ldx, ldc, sm_count, stream);
 }
 
 // A product of many rows with an activation in the epilogue of the persistent kernel (bf16 out):

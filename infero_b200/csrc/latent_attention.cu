@@ -17,6 +17,8 @@
 //   page, the plain query parts to q_plain (the element type of the step) and the rotated ones to q_rot (float32).
 // attention (this file: the any-type kernel, one warp per (token, head); keys in ascending chunks of 32 aligned to
 //   absolute positions, running maximum and sum in 32-bit, so a token's arithmetic depends on its own position only).
+//   With a window W a query at position p sees the keys p - W + 1 .. p; with sinks (one number per head) the softmax's
+//   denominator has one more term exp(sink) without a value.
 // finish: out[t, n * V + v] = val[n, t, v] * sigmoid(gate[t, n]).
 #include "common.cuh"
 #include <math_constants.h>
@@ -98,7 +100,8 @@ __global__ void __launch_bounds__(WARPS * 32)
 latent_attention_generic_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_rot, long long head_rows,
                                 T* __restrict__ out, const T* __restrict__ cache, const int* __restrict__ block_table,
                                 int max_blocks, const int* __restrict__ tok_entry, const int* __restrict__ positions,
-                                int tok_first, int n_tokens, int H, int C, int R, int page_size, float scale) {
+                                int tok_first, int n_tokens, int H, int C, int R, int page_size, float scale, int window,
+                                const float* __restrict__ sinks) {
     extern __shared__ float q_s[];                       // [WARPS][C + R]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -113,15 +116,16 @@ latent_attention_generic_kernel(const float* __restrict__ q_lat, const float* __
     const int pos = positions[t];
     const int* table = block_table + (size_t)tok_entry[t] * max_blocks;
 
-    float m = -CUDART_INF_F, l = 0.f;
+    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    float m = sinks ? sinks[n] : -CUDART_INF_F, l = sinks ? 1.f : 0.f;       // a sink counts as a key seen before all others
     float acc[MAX_C / 32];
 #pragma unroll
     for (int i = 0; i < MAX_C / 32; ++i) acc[i] = 0.f;
-    for (int j0 = 0; j0 <= pos; j0 += 32) {
+    for (int j0 = lo / 32 * 32; j0 <= pos; j0 += 32) {
         const int j = j0 + lane;
         long long row = -1;
         float s = -CUDART_INF_F;
-        if (j <= pos) {
+        if (j >= lo && j <= pos) {
             const int page = table[j / page_size];
             if (page >= 0) {
                 row = ((long long)page * page_size + (j % page_size)) * W;
@@ -216,10 +220,11 @@ int infero_latent_prepare(const float* proj, int proj_stride, int q_off, int kv_
 
 // q_lat float32 [H, head_rows, C] (the plain query parts carried through Wuk^T), q_rot float32 [H, head_rows, R];
 // out [H, head_rows, C] of the cache's type: softmax-weighted sums of the latent rows.  Tokens tok_first .. + n_tokens.
+// window > 0: only that many keys up to the token's own; sinks float32 [H] or null.
 int infero_latent_attention_generic(const float* q_lat, const float* q_rot, long long head_rows, void* out, const void* cache,
                                     int dtype, const int* block_table, int max_blocks, const int* tok_entry,
                                     const int* positions, int tok_first, int n_tokens, int H, int C, int R, int page_size,
-                                    float scale, cudaStream_t stream) {
+                                    float scale, int window, const float* sinks, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     INFERO_REQUIRE(C >= 1 && C <= MAX_C, "latent attention: latent width %d outside 1..%d", C, MAX_C);
     const size_t sh = (size_t)WARPS * (C + R) * sizeof(float);
@@ -228,10 +233,10 @@ int infero_latent_attention_generic(const float* q_lat, const float* q_rot, long
     const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
     if (dtype == INFERO_F32)
         latent_attention_generic_kernel<float><<<blocks, WARPS * 32, sh, stream>>>(q_lat, q_rot, head_rows, (float*)out,
-            (const float*)cache, block_table, max_blocks, tok_entry, positions, tok_first, n_tokens, H, C, R, page_size, scale);
+            (const float*)cache, block_table, max_blocks, tok_entry, positions, tok_first, n_tokens, H, C, R, page_size, scale, window, sinks);
     else
         latent_attention_generic_kernel<bf16><<<blocks, WARPS * 32, sh, stream>>>(q_lat, q_rot, head_rows, (bf16*)out,
-            (const bf16*)cache, block_table, max_blocks, tok_entry, positions, tok_first, n_tokens, H, C, R, page_size, scale);
+            (const bf16*)cache, block_table, max_blocks, tok_entry, positions, tok_first, n_tokens, H, C, R, page_size, scale, window, sinks);
     return infero_check_launch("latent_attention_generic");
 }
 

@@ -12,6 +12,9 @@
 // C result columns, so the result tile of 16 x C/2 (or C/4) stays in registers.  Key tiles start at multiples of 32 of the absolute position, so what is
 // computed for a token does not depend on how its prompt was cut.
 //
+// With a window every row has a lowest key too, and the ranges start at the tile of the first row's lowest key; a learned sink
+// per head is one more term of the rows' sums, added where a row's result is divided by its sum.
+//
 // Single tokens with long contexts are cut into `splits` ranges of keys, one CTA each; every CTA leaves its
 // maximum, sum and unnormalised result, and a second kernel adds them up in ascending order.
 #include "attn_common.cuh"
@@ -34,7 +37,7 @@ latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_r
                   const bf16* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
                   const int* __restrict__ entry_q_start, const int* __restrict__ entry_q_len,
                   const int* __restrict__ entry_pos0, int entry_first, int n_entries, int TQ, int HC, int H, int R,
-                  int page_size, float scale_log2, int chunk, int splits) {
+                  int page_size, float scale_log2, int chunk, int splits, int window, const float* __restrict__ sinks) {
     constexpr int ROWS = ROWG * 16, NT = ROWG * NW * 32, CW = C / NW, NO = CW / 8;
     constexpr int KW = KT / NW, NTW = KW / 8;              // keys, and n-tiles of 8 keys, whose scores a warp forms
     const int W = C + R, LD = W + 8;                       // padded row of a tile, in elements
@@ -67,7 +70,9 @@ latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_r
     const int n_tq = min(TQ, q_len - t0);
     const int head0 = blockIdx.y * HC;
     const int split = blockIdx.z;
-    const int k_lo = split * chunk;
+    // (the first of the tile's tokens sees the lowest key)
+    const int k_base = window > 0 ? max(0, pos_first - window + 1) / KT * KT : 0;
+    const int k_lo = k_base + split * chunk;
     const int k_hi = min(pos_first + n_tq, splits > 1 ? k_lo + chunk : 0x7fffffff);     // one past the last key
     const int* table = block_table + (size_t)e * max_blocks;
 
@@ -128,6 +133,7 @@ latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_r
     const int g = lane >> 2, cq = lane & 3, mi = lane >> 3;
     const int row_a = rg * 16 + g, row_b = row_a + 8;
     const int hi0 = pos_first + row_a / HC, hi1 = pos_first + row_b / HC;      // the last key each of the two rows sees
+    const int lo0 = window > 0 ? hi0 - window + 1 : 0, lo1 = window > 0 ? hi1 - window + 1 : 0;     // and the first
 
     for (int kt = 0; kt < n_tiles; ++kt) {
         cp_async_wait<STAGES - 2>();
@@ -201,8 +207,8 @@ latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_r
             for (int x = 0; x < 2; ++x) {
                 const int j = key0 + part * KW + nt * 8 + cq * 2 + x;
                 const bool in = j >= k_lo && j < k_hi;
-                const float a = (in && j <= hi0) ? s[nt][x] * scale_log2 : -CUDART_INF_F;
-                const float b = (in && j <= hi1) ? s[nt][2 + x] * scale_log2 : -CUDART_INF_F;
+                const float a = (in && j >= lo0 && j <= hi0) ? s[nt][x] * scale_log2 : -CUDART_INF_F;
+                const float b = (in && j >= lo1 && j <= hi1) ? s[nt][2 + x] * scale_log2 : -CUDART_INF_F;
                 s[nt][x] = a, s[nt][2 + x] = b;
                 mx0 = fmaxf(mx0, a), mx1 = fmaxf(mx1, b);
             }
@@ -286,7 +292,7 @@ latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_r
         const int t = tok0 + tq;
         if (splits == 1) {
             bf16* dst = out + ((size_t)n * head_rows + t) * C + part * CW;
-            const float inv = 1.0f / l[x];
+            const float inv = 1.0f / (sinks ? l[x] + exp2f(sinks[n] - m[x]) : l[x]);
 #pragma unroll
             for (int i = 0; i < NO; ++i)
                 *reinterpret_cast<uint32_t*>(dst + i * 8 + cq * 2) = pack_bf16(o[i][2 * x] * inv, o[i][2 * x + 1] * inv);
@@ -307,7 +313,7 @@ latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_r
 constexpr int MAX_SPLITS = 64;
 __global__ void __launch_bounds__(256)
 latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
-                    long long head_rows, int H, int C, int splits) {
+                    long long head_rows, int H, int C, int splits, const float* __restrict__ sinks) {
     __shared__ float w_s[MAX_SPLITS];
     __shared__ float inv_s;
     const int t = blockIdx.x / H, n = blockIdx.x % H;
@@ -322,7 +328,8 @@ latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ 
         const float w0 = m0 == -CUDART_INF_F ? 0.f : exp2f(m0 - M), w1 = m1 == -CUDART_INF_F ? 0.f : exp2f(m1 - M);
         w_s[lane] = w0, w_s[lane + 32] = w1;
         // (the sum in a fixed order: lane by lane through the shuffle tree)
-        const float L = warp_sum(w0 * l0 + w1 * l1);
+        float L = warp_sum(w0 * l0 + w1 * l1);
+        if (sinks) L += exp2f(sinks[n] - M);               // the sink's term, once for all ranges
         if (lane == 0) inv_s = 1.0f / L;
     }
     __syncthreads();
@@ -347,7 +354,7 @@ template <int C, int ROWG, int STAGES, int NW>
 int launch_one(const float* q_lat, const float* q_rot, long long head_rows, bf16* out, float* part_o, float* part_ml,
                const bf16* cache, const int* block_table, int max_blocks, const int* entry_q_start, const int* entry_q_len,
                const int* entry_pos0, int entry_first, int n_entries, int n_tiles, int TQ, int HC, int H, int R,
-               int page_size, float scale, int chunk, int splits, cudaStream_t stream) {
+               int page_size, float scale, int chunk, int splits, int window, const float* sinks, cudaStream_t stream) {
     auto kern = latent_mma_kernel<C, ROWG, STAGES, NW>;
     const int LD = C + R + 8;
     const size_t sh = (size_t)(ROWG * 16 + STAGES * KT) * LD * sizeof(bf16) + (size_t)ROWG * (256 + 64) * 4;
@@ -361,7 +368,7 @@ int launch_one(const float* q_lat, const float* q_rot, long long head_rows, bf16
     const dim3 grid(n_tiles, (H + HC - 1) / HC, splits);
     kern<<<grid, ROWG * NW * 32, sh, stream>>>(q_lat, q_rot, head_rows, out, part_o, part_ml, cache, block_table, max_blocks,
                                           entry_q_start, entry_q_len, entry_pos0, entry_first, n_entries, TQ, HC, H, R,
-                                          page_size, scale * 1.4426950408889634f, chunk, splits);
+                                          page_size, scale * 1.4426950408889634f, chunk, splits, window, sinks);
     return 0;
 }
 
@@ -382,11 +389,13 @@ int infero_latent_mma_heads(int H) { return H <= 16 ? 16 : H <= 32 ? 32 : 64; }
 // single != 0: every entry brings one token (TQ = 1) and the keys are cut into `splits` ranges of `chunk` (a multiple of
 // 32); with splits > 1 part_o float32 [tokens * H * splits * C] and part_ml [tokens * H * splits * 2] are scratch, indexed
 // by the token's row in the step, and the merge runs behind.  Otherwise TQ = 64 / heads per CTA and splits = 1.
+// window > 0: a token sees that many keys up to its own (the ranges then start at the tile of its lowest key); sinks float32
+// [H] (times log2 e) or null: one more term 2^sink of a head's sum.
 int infero_latent_attention_mma(const float* q_lat, const float* q_rot, long long head_rows, void* out, float* part_o,
                                 float* part_ml, const void* cache, const int* block_table, int max_blocks,
                                 const int* entry_q_start, const int* entry_q_len, const int* entry_pos0, int entry_first,
                                 int n_entries, int n_tiles, int single, int H, int C, int R, int page_size, float scale,
-                                int chunk, int splits, cudaStream_t stream) {
+                                int chunk, int splits, int window, const float* sinks, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     INFERO_REQUIRE(infero_latent_mma_supported(C, R), "latent attention: no tensor-core instance for a latent of %d + %d", C, R);
     INFERO_REQUIRE(splits <= MAX_SPLITS, "latent attention: %d ranges of keys, at most %d", splits, MAX_SPLITS);
@@ -399,7 +408,7 @@ int infero_latent_attention_mma(const float* q_lat, const float* q_rot, long lon
 #define GO(C_, ROWG_, ST_)                                                                                              \
     rc = launch_one<C_, ROWG_, ST_, (C_ >= 256 && ROWG_ < 4 ? 4 : 2)>(q_lat, q_rot, head_rows, (bf16*)out, part_o, part_ml, (const bf16*)cache, block_table, \
                                     max_blocks, entry_q_start, entry_q_len, entry_pos0, entry_first, n_entries, n_tiles, TQ, \
-                                    HC, H, R, page_size, scale, chunk, splits, stream)
+                                    HC, H, R, page_size, scale, chunk, splits, window, sinks, stream)
 #define BY_ROWS(C_)                                  \
     do {                                             \
         if (rowg == 1) GO(C_, 1, 2);                 \
@@ -415,7 +424,7 @@ int infero_latent_attention_mma(const float* q_lat, const float* q_rot, long lon
     if (rc) return rc;
     if (splits > 1) {
         // the tokens of the leading single-token entries are the first rows of the step
-        latent_merge_kernel<<<n_tiles * H, C >= 256 ? 256 : 128, 0, stream>>>(part_o, part_ml, (bf16*)out, head_rows, H, C, splits);
+        latent_merge_kernel<<<n_tiles * H, C >= 256 ? 256 : 128, 0, stream>>>(part_o, part_ml, (bf16*)out, head_rows, H, C, splits, sinks);
     }
     return infero_check_launch("latent_attention_mma");
 }

@@ -12,7 +12,10 @@
 //   is formed in 64-bit from a 64-bit table made on the host (any scaling of the frequencies is the host's) and brought
 //   into [-pi, pi] before sincosf; cos and sin are multiplied by `amp`.
 //
-//   values: a projection of their own (v_off >= 0), or the keys as projected, before norm and rotation (v_off < 0).
+//   temperature (temp_every > 0): behind norm and rotation a query at position p is multiplied by
+//           1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+//
+//   values: a projection of their own (v_off >= 0) times v_scale, or the keys as projected, before norm and rotation (v_off < 0).
 //
 // The query goes to q_out in the step's element type, keys and values to the token's page (write_cache; a layer that
 // reads another layer's cache has no key or value columns at all).  One block per token; the row is staged in shared
@@ -33,7 +36,7 @@ qk_prepare_kernel(const float* __restrict__ proj, int proj_stride, int q_off, in
                   const double* __restrict__ freq, int rot, float amp, const int* __restrict__ positions,
                   const int* __restrict__ tok_entry, const int* __restrict__ block_table, int max_blocks, int page_size,
                   T* __restrict__ q_out, int q_stride, T* __restrict__ k_cache, T* __restrict__ v_cache, int write_cache,
-                  int H, int G, int D, int V) {
+                  int H, int G, int D, int V, float temp_coef, float temp_every, float v_scale) {
     extern __shared__ float smem[];
     __shared__ float red[32];
     const int half = rot / 2;
@@ -67,7 +70,7 @@ qk_prepare_kernel(const float* __restrict__ proj, int proj_stride, int q_off, in
         if (v_off >= 0) {
             for (int i = tid; i < G * V; i += THREADS) {
                 const int g = i / V, c = i % V;
-                v_cache[(page_row + (long long)g * page_size) * V + c] = from_f32<T>(row[v_off + i]);
+                v_cache[(page_row + (long long)g * page_size) * V + c] = from_f32<T>(row[v_off + i] * v_scale);
             }
         } else {
             for (int i = tid; i < nk; i += THREADS) {
@@ -123,7 +126,9 @@ qk_prepare_kernel(const float* __restrict__ proj, int proj_stride, int q_off, in
         __syncthreads();
     }
     T* qo = q_out + (size_t)t * q_stride;
-    for (int i = tid; i < nq; i += THREADS) qo[i] = from_f32<T>(buf[i]);
+    float temp = 1.f;
+    if (temp_every > 0.f) temp = fmaf(temp_coef, logf((float)(floor((double)(pos + 1) / (double)temp_every) + 1.0)), 1.f);
+    for (int i = tid; i < nq; i += THREADS) qo[i] = from_f32<T>(buf[i] * temp);
     for (int i = tid; i < nk; i += THREADS) {
         const int g = i / D, c = i % D;
         k_cache[(page_row + (long long)g * page_size) * D + c] = from_f32<T>(buf[nq + i]);
@@ -170,7 +175,8 @@ int infero_qk_prepare(const float* proj, int proj_stride, int q_off, int k_off, 
                       const void* q_norm_w, const void* k_norm_w, int norm_w_dtype, float eps, const double* freq,
                       int rot, float amp, const int* positions, const int* tok_entry, const int* block_table,
                       int max_blocks, int page_size, void* q_out, int q_stride, void* k_cache, void* v_cache, int dtype,
-                      int write_cache, int n_tokens, int H, int G, int D, int V, cudaStream_t stream) {
+                      int write_cache, int n_tokens, int H, int G, int D, int V, float temp_coef, float temp_every, float v_scale,
+                      cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     INFERO_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= D, "qk_prepare: %d rotated coordinates of %d", rot, D);
     INFERO_REQUIRE(norm_mode >= 0 && norm_mode <= 3, "qk_prepare: norm mode %d", norm_mode);
@@ -185,7 +191,7 @@ int infero_qk_prepare(const float* proj, int proj_stride, int q_off, int k_off, 
         k<<<n_tokens, THREADS, smem, stream>>>(proj, proj_stride, q_off, k_off, v_off, norm_mode, q_norm_w, k_norm_w,    \
                                                norm_w_dtype, eps, freq, rot, amp, positions, tok_entry, block_table,      \
                                                max_blocks, page_size, (T*)q_out, q_stride, (T*)k_cache, (T*)v_cache,      \
-                                               write_cache, H, G, D, V);                                                  \
+                                               write_cache, H, G, D, V, temp_coef, temp_every, v_scale);                                                  \
     } while (0)
     if (dtype == INFERO_F32) LAUNCH(float);
     else LAUNCH(bf16);

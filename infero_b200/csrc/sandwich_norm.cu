@@ -5,7 +5,8 @@
 //   y   = sum of the pending sublayer's result: one 32-bit array or several partial sums (the split-K products of the
 //         few-token matrix kernel), plus a bias; or two such results side by side, z = scale * sum_b rms(y_b) * w_b
 //   x  += rms(z) * w_post            (w_post null: x += z)
-//   h   = rms(x) * w_pre             (the next sublayer's input, or the rows the output product wants)
+//   h   = rms(x) * w_pre             (the next sublayer's input, or the rows the output product wants; w_pre null: h = x, what
+//                                     sublayers without a norm in front read; out null: h is not wanted at all)
 //
 // with rms(v) = v / sqrt(mean(v^2) + eps).  The weights come as what multiplies (a norm whose stored weight is the
 // distance from one is made so at load time).  In steps of single tokens the input convolution below is part of the same
@@ -184,15 +185,18 @@ sandwich_norm_kernel(float* __restrict__ x, const Branch b0, const Branch b1, in
 #pragma unroll
         for (int k = 0; k < VEC; ++k) sx = fmaf(v[k], v[k], sx);
     }
-    const float rx = 1.0f / sqrtf(block_sum2(sx, 0.f, red).x * inv_d + pre_eps);
+    if (!out) return;
+    const float rx = w_pre ? 1.0f / sqrtf(block_sum2(sx, 0.f, red).x * inv_d + pre_eps) : 1.f;
     TO* orow = out + (size_t)r * d;
     float* tail = conv.w ? conv.state + (long long)conv.entry_slot[conv.tok_entry[src]] * conv.state_stride : nullptr;
     for (int i = i0; i < d; i += step) {
         float h[VEC], w[VEC];
         load_v<VEC>(z + i, h);
-        load_v<VEC>(w_pre + i, w);
+        if (w_pre) {
+            load_v<VEC>(w_pre + i, w);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) h[k] = h[k] * rx * w[k];
+            for (int k = 0; k < VEC; ++k) h[k] = h[k] * rx * w[k];
+        }
         if (conv.w) {
             float acc[VEC], old[VEC];
 #pragma unroll
@@ -249,7 +253,7 @@ sandwich_rows_kernel(float* __restrict__ x, const Branch b0, const Branch b1, fl
     const float inv_d = 1.0f / (float)d;
     float wq[4] = {0.f, 0.f, 0.f, 0.f}, wp[4] = {0.f, 0.f, 0.f, 0.f};
     if (mine) {
-        load4(w_pre + i, wq);
+        if (w_pre) load4(w_pre + i, wq);
         if (NB > 0 && w_post) load4(w_post + i, wp);
     }
     pdl_wait();
@@ -298,10 +302,12 @@ sandwich_rows_kernel(float* __restrict__ x, const Branch b0, const Branch b1, fl
         float sx = 0.f;
 #pragma unroll
         for (int k = 0; k < 4; ++k) sx = fmaf(v[k], v[k], sx);
-        const float rx = 1.0f / sqrtf(block_sum(sx, red) * inv_d + pre_eps);
-        if (!mine) continue;
+        const float rx = w_pre ? 1.0f / sqrtf(block_sum(sx, red) * inv_d + pre_eps) : 1.f;
+        if (!mine || !out) continue;
+        if (w_pre) {
 #pragma unroll
-        for (int k = 0; k < 4; ++k) v[k] = v[k] * rx * wq[k];
+            for (int k = 0; k < 4; ++k) v[k] = v[k] * rx * wq[k];
+        }
         if (conv.w) {
             float* tail = conv.state + (long long)conv.entry_slot[conv.tok_entry[src]] * conv.state_stride + i;
             float acc[4] = {0.f, 0.f, 0.f, 0.f}, old[4], w[4];
@@ -440,6 +446,8 @@ int infero_sandwich_norm(float* x, const float* y0, int splits0, long long strid
                          cudaStream_t stream) {
     if (n_rows == 0) return 0;
     INFERO_REQUIRE(d > 0 && (size_t)d * 8 <= 200 * 1024, "sandwich_norm: width %d not supported", d);
+    INFERO_REQUIRE(w_pre || !conv_w, "sandwich_norm: a convolution needs a normed input");
+    INFERO_REQUIRE(out || !w_pre, "sandwich_norm: a norm without a place for its result");
     INFERO_REQUIRE(!y1 || y0, "sandwich_norm: a second branch without a first");
     INFERO_REQUIRE(!conv_w || (taps >= 1 && taps <= MAX_TAPS && !rows), "sandwich_norm: %d taps outside 1..%d", taps, MAX_TAPS);
     const Branch b0 = {y0, bias0, w0, stride0, splits0}, b1 = {y1, bias1, w1, stride1, splits1};

@@ -296,17 +296,19 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                       n_heads: int, n_kv: int, head_dim: int, page_size: int, window: Optional[int],
                       scale: float, value_dim: int = 0, sink: bool = False,
                       slopes: Optional[torch.Tensor] = None, rel: Optional[torch.Tensor] = None,
-                      cross: bool = False) -> None:
+                      cross: bool = False, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
     """q: [T, >= H*D] view (row stride free), out [T, H*V] with V = ``value_dim`` (0: the keys' width).  ``sink``: one
     more term exp(0) in the softmax's sum, without a value.  ``slopes`` float32 [H]: head h's score loses slopes[h]
     times the distance between the query and the key.  ``rel`` float32 [H, L]: head h's score gains rel[h, min(distance,
     L - 1)].  ``cross``: every head's weights meet the values of every kv head, out float32 [T, G * H * V] (row
-    c H + h: head h over kv head c's values)."""
+    c H + h: head h over kv head c's values).  ``sinks`` float32 [H]: one more term exp(sinks[h]) in the sum, without a
+    value.  ``softcap`` > 0: a scaled score s becomes softcap tanh(s / softcap) before any bias."""
     T = q.shape[0]
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == k_cache.dtype
     assert out.dtype == (torch.float32 if cross else q.dtype)
     assert out.shape[1] == n_heads * (value_dim or head_dim) * (n_kv if cross else 1)
     assert rel is None or (rel.dtype == torch.float32 and rel.is_contiguous() and rel.dim() == 2 and rel.shape[0] == n_heads)
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == n_heads)
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.is_contiguous() and slopes.numel() == n_heads)
     _check(lib().infero_attention_generic_rel(_ptr(q), c_int(q.stride(0)), _ptr(out), c_int(out.stride(0)),
                                              _ptr(k_cache), _ptr(v_cache), c_int(_dt(q)),
@@ -316,6 +318,7 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                                              c_int(value_dim or head_dim), c_int(page_size), c_int(window or 0),
                                              c_float(scale), c_int(1 if sink else 0), _ptr(slopes), _ptr(rel),
                                              c_int(rel.shape[1] if rel is not None else 0), c_int(1 if cross else 0),
+                                             _ptr(sinks), c_float(softcap),
                                              _stream()))
 
 

@@ -57,12 +57,13 @@ def _rel_args(rel):
 
 def decode(q, out, k_cache, v_cache, table, tok_entry, positions, tok_first: int, n_tok: int, n_heads: int,
            n_kv: int, head_dim: int, page_size: int, window: Optional[int], scale: float, chunk: int,
-           n_splits: int, sink: bool = False, slopes=None, rel=None, cross: bool = False) -> None:
+           n_splits: int, sink: bool = False, slopes=None, rel=None, cross: bool = False, sinks=None, softcap: float = 0.0) -> None:
     """``rel`` (float32 [H, L], times log2 e) and ``cross``: see ``paged_attention_cross``.  ``sink``: one more term exp(0) in the softmax's sum, added where the splits of a row are merged.  ``slopes``
-    (float32 [H]): head h's score loses slopes[h] times the distance between the query and the key."""
+    (float32 [H]): head h's score loses slopes[h] times the distance between the query and the key.  ``sinks`` (float32 [H],
+    times log2 e): one more term 2^sinks[h] of head h's sum.  ``softcap`` > 0: scaled scores are soft-capped."""
     need = int(lib_scratch(n_tok, n_heads * (n_kv if cross else 1), head_dim, n_splits))
     scratch = torch.empty(need // 4, dtype=torch.float32, device=q.device)
-    more = (_ptr(slopes), *_rel_args(rel), c_int(1 if cross else 0))
+    more = (_ptr(slopes), *_rel_args(rel), c_int(1 if cross else 0), _ptr(sinks), c_float(softcap))
     if lib().infero_attn_decode_tma_supported(c_int(head_dim), c_int(page_size)) and k_cache.is_contiguous() \
             and v_cache.is_contiguous():
         _check(lib().infero_attn_decode_tma_ex(
@@ -110,14 +111,15 @@ def lib_scratch(n_tok, n_heads, head_dim, n_splits) -> int:
 
 def prefill(q, out, k_cache, v_cache, table, entry_q_start, entry_q_len, entry_pos0, n_entries: int,
             first_entry: int, n_tiles: int, n_heads: int, n_kv: int, head_dim: int, page_size: int,
-            window: Optional[int], scale: float, sink: bool = False, slopes=None, rel=None, cross: bool = False) -> None:
+            window: Optional[int], scale: float, sink: bool = False, slopes=None, rel=None, cross: bool = False, sinks=None,
+            softcap: float = 0.0) -> None:
     _check(lib().infero_attn_prefill_ex(_ptr(q), c_int(q.stride(0)), _ptr(out), c_int(out.stride(0)), _ptr(k_cache),
                                           _ptr(v_cache), _ptr(_i32(table, "block_table")), c_int(table.shape[1]),
                                           _ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")),
                                           _ptr(_i32(entry_pos0, "entry_pos0")), c_int(n_entries), c_int(first_entry),
                                           c_int(n_tiles), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(page_size),
                                           c_int(window or 0), c_float(scale), c_int(1 if sink else 0), _ptr(slopes),
-                                          *_rel_args(rel), c_int(1 if cross else 0), _stream()))
+                                          *_rel_args(rel), c_int(1 if cross else 0), _ptr(sinks), c_float(softcap), _stream()))
 
 
 def prefill_tc_supported(q, out, head_dim: int, page_size: int) -> bool:
@@ -128,7 +130,8 @@ def prefill_tc_supported(q, out, head_dim: int, page_size: int) -> bool:
 
 def prefill_tc(q, out, k_cache, v_cache, table, entry_q_start, entry_q_len, entry_pos0, n_entries: int,
                first_entry: int, n_tiles: int, n_heads: int, n_kv: int, head_dim: int, page_size: int,
-               window: Optional[int], scale: float, sink: bool = False, slopes=None, rel=None, cross: bool = False) -> None:
+               window: Optional[int], scale: float, sink: bool = False, slopes=None, rel=None, cross: bool = False, sinks=None,
+            softcap: float = 0.0) -> None:
     """The tcgen05 kernel: 128 query rows per block (n_tiles counts blocks of 128)."""
     _check(lib().infero_attn_prefill_tc_ex(
         _ptr(q), c_int(q.stride(0)), c_int(q.shape[0]), _ptr(out), c_int(out.stride(0)), _ptr(k_cache), _ptr(v_cache),
@@ -136,7 +139,7 @@ def prefill_tc(q, out, k_cache, v_cache, table, entry_q_start, entry_q_len, entr
         _ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")),
         _ptr(_i32(entry_pos0, "entry_pos0")), c_int(n_entries), c_int(first_entry), c_int(n_tiles), c_int(n_heads),
         c_int(n_kv), c_int(head_dim), c_int(page_size), c_int(window or 0), c_float(scale), c_int(1 if sink else 0),
-        _ptr(slopes), *_rel_args(rel), c_int(1 if cross else 0), _stream()))
+        _ptr(slopes), *_rel_args(rel), c_int(1 if cross else 0), _ptr(sinks), c_float(softcap), _stream()))
 
 
 def shape_of_batch(q_lens: Sequence[int], pos0: Sequence[int]):
@@ -156,18 +159,21 @@ def shape_of_batch(q_lens: Sequence[int], pos0: Sequence[int]):
 def attention_any(q, out, k_cache, v_cache, table, tok_entry, positions, n_heads: int, n_kv: int, head_dim: int,
                   page_size: int, window: Optional[int], scale: float, q_lens: Sequence[int], pos0: Sequence[int],
                   entry_q_start=None, entry_q_len=None, entry_pos0=None, kv_bound: Optional[int] = None,
-                  batch_shape=None, sink: bool = False, slopes=None, rel=None, rel_log2=None, cross: bool = False) -> None:
+                  batch_shape=None, sink: bool = False, slopes=None, rel=None, rel_log2=None, cross: bool = False, sinks=None,
+                  sinks_log2=None, softcap: float = 0.0) -> None:
     """q: [T, >= H*D] view with rotated queries in front (row stride free); out [T, H*D].
     ``q_lens`` / ``pos0`` are the host copies of each request's new-token count and cached
     length; the device copies are made here when the caller has none.  ``kv_bound``: plan the
     decode splits for this many visible keys instead of what the batch holds now (a captured
     step is replayed while its requests grow).  ``slopes`` (float32 [H]): a distance bias per head.
     ``rel`` (float32 [H, L]; ``rel_log2``: the same times log2 e, for the bf16 kernels) and ``cross``: see
-    ``paged_attention_cross``; out [T, G*H*D] then, float32 where the any-type kernel runs."""
+    ``paged_attention_cross``; out [T, G*H*D] then, float32 where the any-type kernel runs.  ``sinks`` (float32 [H];
+    ``sinks_log2``: the same times log2 e) and ``softcap``: see ``paged_attention_ex``."""
     if q.dtype != torch.bfloat16 or not mma_supported(head_dim, page_size):
         attention_generic(q, out, k_cache, v_cache, table, tok_entry, positions, n_heads, n_kv, head_dim,
-                          page_size, window, scale, sink=sink, slopes=slopes, rel=rel, cross=cross)
+                          page_size, window, scale, sink=sink, slopes=slopes, rel=rel, cross=cross, sinks=sinks, softcap=softcap)
         return
+    more = dict(sink=sink, slopes=slopes, rel=rel_log2, cross=cross, sinks=sinks_log2, softcap=softcap)
     sides = n_kv if cross else 1
     E = len(q_lens)
     if batch_shape is None:
@@ -179,7 +185,7 @@ def attention_any(q, out, k_cache, v_cache, table, tok_entry, positions, n_heads
             vis = min(vis, window + 15)
         chunk, splits = plan_decode(n_dec, n_kv * sides, n_heads // n_kv, vis)
         decode(q, out, k_cache, v_cache, table, tok_entry, positions, 0, n_dec, n_heads, n_kv, head_dim,
-               page_size, window, scale, chunk, splits, sink=sink, slopes=slopes, rel=rel_log2, cross=cross)
+               page_size, window, scale, chunk, splits, **more)
     if n_dec < E:
         if entry_q_len is None:
             dev = q.device
@@ -192,11 +198,11 @@ def attention_any(q, out, k_cache, v_cache, table, tok_entry, positions, n_heads
         if prefill_tc_supported(q, out, head_dim, page_size) and k_cache.is_contiguous() and v_cache.is_contiguous():
             n_tiles = tiles_128
             prefill_tc(q, out, k_cache, v_cache, table, entry_q_start, entry_q_len, entry_pos0, E, n_dec, n_tiles,
-                       n_heads, n_kv, head_dim, page_size, window, scale, sink=sink, slopes=slopes, rel=rel_log2, cross=cross)
+                       n_heads, n_kv, head_dim, page_size, window, scale, **more)
             return
         n_tiles = tiles_mma
         prefill(q, out, k_cache, v_cache, table, entry_q_start, entry_q_len, entry_pos0, E, n_dec, n_tiles,
-                n_heads, n_kv, head_dim, page_size, window, scale, sink=sink, slopes=slopes, rel=rel_log2, cross=cross)
+                n_heads, n_kv, head_dim, page_size, window, scale, **more)
 
 
 def paged_attention(ctx, qkv, out, kv, table, n_heads, n_kv, head_dim, window, scale, sink: bool = False, slopes=None) -> None:
@@ -218,19 +224,32 @@ def _batch_shape(ctx):
     return memo
 
 
+LOG2E = 1.4426950408889634
+
+
 def paged_attention_ex(ctx, q, out, kv, table, n_heads, n_kv, head_dim, value_dim, window, scale, sink: bool,
-                       slopes=None, rel=None) -> None:
-    """Attention with values of their own width and, optionally, a sink (one more term exp(0) in the softmax's sum, without
-    a value) or a distance bias (``slopes`` float32 [H]: head h's score loses slopes[h] times the distance to the key).
-    q [T, H*D] rotated queries; out [T, H*V].  Equal widths take the same kernels as ``paged_attention`` (the sink is a
-    term added to the sum where a row's result is divided by it, the bias a term added to a score where it is masked);
-    values of another width than the keys, and a bias by a table of distances (``rel`` float32 [H, L]), run on the any-type
-    kernel."""
-    if value_dim == head_dim and rel is None:
-        paged_attention(ctx, q, out, kv, table, n_heads, n_kv, head_dim, window, scale, sink=sink, slopes=slopes)
+                       slopes=None, rel=None, rel_log2=None, sinks=None, sinks_log2=None, softcap: float = 0.0) -> None:
+    """Attention with values of their own width and what a layer may want besides: a sink (one more term exp(0) in the
+    softmax's sum, without a value), learned sinks (``sinks`` float32 [H]: exp(sinks[h])), a distance bias (``slopes`` float32
+    [H]: head h's score loses slopes[h] times the distance to the key; or ``rel`` float32 [H, L]: it gains rel[h, min(distance,
+    L - 1)]), a soft cap of the scaled score ahead of any bias (``softcap`` c > 0: c tanh(s / c)).
+    q [T, H*D] rotated queries; out [T, H*V].  Equal widths take the same kernels as ``paged_attention`` (sinks are
+    terms added to the sum where a row's result is divided by it, biases terms added to a score where it is masked);
+    values of another width than the keys run on the any-type kernel.  ``rel_log2``, ``sinks_log2``: the same times log2 e,
+    as the bf16 kernels take them (made here when absent)."""
+    signed = rel is not None or slopes is not None or softcap > 0      # what the bf16 kernels want a positive scale for
+    if value_dim == head_dim and (scale > 0 or not signed):
+        if rel is not None and rel_log2 is None:
+            rel_log2 = rel * LOG2E
+        if sinks is not None and sinks_log2 is None:
+            sinks_log2 = sinks * LOG2E
+        attention_any(q, out, kv.k, kv.v, table, ctx.tok_entry, ctx.positions, n_heads, n_kv, head_dim, kv.page_size, window, scale,
+                      ctx.h_q_len, ctx.h_pos0, ctx.entry_q_start, ctx.entry_q_len, ctx.entry_pos0,
+                      kv_bound=getattr(ctx, "kv_bound", None), batch_shape=_batch_shape(ctx), sink=sink, slopes=slopes, rel=rel,
+                      rel_log2=rel_log2, sinks=sinks, sinks_log2=sinks_log2, softcap=softcap)
         return
     attention_generic(q, out, kv.k, kv.v, table, ctx.tok_entry, ctx.positions, n_heads, n_kv, head_dim, kv.page_size,
-                      window, scale, value_dim=value_dim, sink=sink, slopes=slopes, rel=rel)
+                      window, scale, value_dim=value_dim, sink=sink, slopes=slopes, rel=rel, sinks=sinks, softcap=softcap)
 
 
 def paged_attention_cross(ctx, q, kv, table, n_heads, n_kv, head_dim, value_dim, window, scale, rel=None,

@@ -82,21 +82,25 @@ def per_head_product(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_rows
 
 
 def attention(ctx, q_lat: torch.Tensor, q_rot: torch.Tensor, out: torch.Tensor, kv, table, n_tokens: int, H: int, C: int,
-              R: int, scale: float) -> None:
+              R: int, scale: float, window: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
+              sinks_log2: Optional[torch.Tensor] = None) -> None:
     """Causal softmax attention of every token over its request's cached latent rows: q_lat float32 [H, rows, C],
-    q_rot float32 [H, rows, R], out [H, rows, C] of the cache's type."""
+    q_rot float32 [H, rows, R], out [H, rows, C] of the cache's type.  ``window``: a token sees that many keys up to its own.
+    ``sinks`` float32 [H] (``sinks_log2``: times log2 e, made here when absent): one more term exp(sinks[h]) in head h's sum,
+    without a value."""
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == H)
     cache = kv.k
     rows = q_lat.shape[1]
     assert q_lat.dtype == torch.float32 and q_rot.dtype == torch.float32 and q_lat.is_contiguous() and q_rot.is_contiguous()
     assert out.dtype == cache.dtype and out.is_contiguous() and tuple(out.shape) == (H, rows, C) and cache.is_contiguous()
     from . import latent_mma
-    if latent_mma.run(ctx, q_lat, q_rot, out, kv, table, n_tokens, H, C, R, scale):
+    if latent_mma.run(ctx, q_lat, q_rot, out, kv, table, n_tokens, H, C, R, scale, window, sinks, sinks_log2):
         return
     _check(lib().infero_latent_attention_generic(
         _ptr(q_lat), _ptr(q_rot), c_longlong(rows), _ptr(out), _ptr(cache), c_int(_dt(cache)),
         _ptr(_i32(table, "block_table")), c_int(table.shape[1]), _ptr(_i32(ctx.tok_entry, "tok_entry")),
         _ptr(_i32(ctx.positions, "positions")), c_int(0), c_int(n_tokens), c_int(H), c_int(C), c_int(R),
-        c_int(kv.page_size), c_float(scale), _stream()))
+        c_int(kv.page_size), c_float(scale), c_int(window or 0), _ptr(sinks), _stream()))
 
 
 def finish(val: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, n_tokens: int, H: int, V: int) -> None:

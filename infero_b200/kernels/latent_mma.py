@@ -31,13 +31,16 @@ def plan_splits(n_tok: int, head_blocks: int, visible: int, sms: int):
     return chunk, -(-visible // chunk)
 
 
-def run(ctx, q_lat, q_rot, out, kv, table, n_tokens, H, C, R, scale) -> bool:
+def run(ctx, q_lat, q_rot, out, kv, table, n_tokens, H, C, R, scale, window=None, sinks=None, sinks_log2=None) -> bool:
     cache = kv.k
     if not ENABLED or cache.dtype != torch.bfloat16 or not supported(C, R) or getattr(ctx, "h_q_len", None) is None:
         return False
     from .attention import _batch_shape
     from .tc_gemm import sm_count
     n_dec, vis_now, _, _ = _batch_shape(ctx)
+    if sinks is not None and sinks_log2 is None:
+        sinks_log2 = sinks * 1.4426950408889634
+    more = (c_int(window or 0), _ptr(sinks_log2))
     E = ctx.n_entries
     HC = int(lib().infero_latent_mma_heads(c_int(H)))
     rows = q_lat.shape[1]
@@ -45,6 +48,8 @@ def run(ctx, q_lat, q_rot, out, kv, table, n_tokens, H, C, R, scale) -> bool:
               _ptr(_i32(ctx.entry_q_len, "entry_q_len")), _ptr(_i32(ctx.entry_pos0, "entry_pos0")))
     if n_dec:
         vis = vis_now if getattr(ctx, "kv_bound", None) is None else int(ctx.kv_bound)
+        if window:
+            vis = min(vis, int(window) + 31)             # (ranges start at the tile of the lowest key seen)
         chunk, splits = plan_splits(n_dec, -(-H // HC), max(vis, 1), sm_count(q_lat.device))
         part_o = part_ml = None
         launches["single"] += 1
@@ -55,12 +60,12 @@ def run(ctx, q_lat, q_rot, out, kv, table, n_tokens, H, C, R, scale) -> bool:
         _check(lib().infero_latent_attention_mma(_ptr(q_lat), _ptr(q_rot), c_longlong(rows), _ptr(out), _ptr(part_o), _ptr(part_ml),
                                                  *common, c_int(0), c_int(n_dec), c_int(n_dec), c_int(1), c_int(H), c_int(C),
                                                  c_int(R), c_int(kv.page_size), c_float(scale), c_int(chunk), c_int(splits),
-                                                 _stream()))
+                                                 *more, _stream()))
     if n_dec < E:
         TQ = 64 // HC
         launches["tiled"] += 1
         tiles = sum(-(-int(n) // TQ) for n in ctx.h_q_len[n_dec:])
         _check(lib().infero_latent_attention_mma(_ptr(q_lat), _ptr(q_rot), c_longlong(rows), _ptr(out), _ptr(None), _ptr(None),
                                                  *common, c_int(n_dec), c_int(E), c_int(tiles), c_int(0), c_int(H), c_int(C),
-                                                 c_int(R), c_int(kv.page_size), c_float(scale), c_int(0), c_int(1), _stream()))
+                                                 c_int(R), c_int(kv.page_size), c_float(scale), c_int(0), c_int(1), *more, _stream()))
     return True

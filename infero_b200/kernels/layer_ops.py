@@ -266,14 +266,20 @@ def _product_in(v):
     return v, _dt(v), 1, 0, tuple(v.shape)
 
 
-def glu_act(gate_up, out: torch.Tensor, act=None) -> None:
+def glu_act(gate_up, out: torch.Tensor, act=None, bias: Optional[torch.Tensor] = None) -> None:
     """out[t, j] = glu(g[t, 2j], g[t, 2j + 1]) for g = gate_up (a tensor or ``Partials``; gate and up alternate along a
-    row); ``act`` = (kind, limit, alpha), None: silu(g) * u."""
+    row); ``act`` = (kind, limit, alpha), None: silu(g) * u; ``bias`` float32 [2 ff] is added to g first (``Partials`` bring
+    their own)."""
     T, ff = out.shape
+    if getattr(gate_up, "bias", None) is not None:
+        from . import Partials
+        assert bias is None
+        gate_up, bias = Partials(gate_up.data), gate_up.bias
+    assert bias is None or bias.numel() == 2 * ff
     data, dt, splits, stride, shape = _product_in(gate_up)
     assert shape == (T, 2 * ff) and out.is_contiguous()
     _check(lib().infero_glu_act(_ptr(data), c_int(dt), c_int(splits), c_longlong(stride), _ptr(out), c_int(_dt(out)), c_int(T),
-                                c_int(ff), *_act_args(act), _stream()))
+                                c_int(ff), *_act_args(act), _ptr(_f32(bias, "bias")), _stream()))
 
 
 def relu2(v, out: torch.Tensor) -> None:
@@ -337,12 +343,15 @@ def streams_fill(x: torch.Tensor, xs: torch.Tensor) -> None:
 # ---- normed attention, gated linear recurrence (csrc/qk_prepare.cu, rglru.cu) ------------------------------------
 def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, norm_mode: int, q_norm_w, k_norm_w, eps: float,
                freq64: Optional[torch.Tensor], amp: float, positions, tok_entry, block_table, page_size: int,
-               q_out: torch.Tensor, k_cache, v_cache, H: int, G: int, D: int, V: int, write_cache: bool = True) -> None:
+               q_out: torch.Tensor, k_cache, v_cache, H: int, G: int, D: int, V: int, write_cache: bool = True,
+               temperature=None, v_scale: float = 1.0) -> None:
     """From the 32-bit product row of every token (``proj`` [T, >= ...], columns ``q_off`` / ``k_off`` / ``v_off``; a
     negative ``v_off``: the values are the keys as projected) to normed, rotated queries in ``q_out`` [T, H*D] and keys and
     values in the token's page.  ``norm_mode`` 0 none, 1 weighted RMS over the whole projection before the rotation,
     2 unit RMS per head after it, 3 weighted RMS per head before it (weights of D numbers shared by the heads).
-    ``freq64`` float64 [rot/2] (None: no rotation), ``amp`` multiplies cos and sin."""
+    ``freq64`` float64 [rot/2] (None: no rotation), ``amp`` multiplies cos and sin.  ``temperature`` = (coef, every): a
+    query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at the end.  ``v_scale`` multiplies values
+    of a projection of their own."""
     T = proj.shape[0]
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and q_out.stride(1) == 1 and q_out.shape == (T, H * D)
     rot = 0
@@ -364,7 +373,8 @@ def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, norm_mode
         c_float(amp), _ptr(_i32(positions, "positions")), _ptr(_i32(tok_entry, "tok_entry")),
         _ptr(_i32(block_table, "block_table")), c_int(block_table.shape[1]), c_int(page_size), _ptr(q_out),
         c_int(q_out.stride(0)), _ptr(k_cache if write_cache else None), _ptr(v_cache if write_cache else None),
-        c_int(_dt(q_out)), c_int(1 if write_cache else 0), c_int(T), c_int(H), c_int(G), c_int(D), c_int(V), _stream()))
+        c_int(_dt(q_out)), c_int(1 if write_cache else 0), c_int(T), c_int(H), c_int(G), c_int(D), c_int(V),
+        c_float(temperature[0] if temperature else 0.0), c_float(temperature[1] if temperature else 0.0), c_float(v_scale), _stream()))
 
 
 def head_gate(a: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, H: int, V: int, scale: float = 1.0) -> None:
@@ -508,17 +518,18 @@ def _branch(v, shape):
     return v, 1, 0, None
 
 
-def sandwich_norm(x: torch.Tensor, delta, weight: torch.Tensor, eps: float, out: torch.Tensor,
+def sandwich_norm(x: torch.Tensor, delta, weight: Optional[torch.Tensor], eps: float, out: Optional[torch.Tensor],
                   rows: Optional[torch.Tensor] = None, conv=None) -> None:
     """x += rms(z) * w for a pending ``NormedDelta`` (None: x is left as it is; a plain 32-bit tensor or ``Partials`` is
-    added as it is), then out = rms(x) * weight.  With ``rows`` only those rows are worked on and x is left as it is.
+    added as it is), then out = rms(x) * weight (no weight: out = x; no out: nothing more).  With ``rows`` only those rows are worked on and x is left as it is.
     ``conv`` = (weights [taps, d], state [slots, (taps - 1) d], tok_entry, entry_slot): in a step of single tokens, out
     becomes out + the convolution of it over the requests' earlier rows, and the state moves on."""
     from . import BranchSum, NormedDelta
     d = x.shape[1]
-    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape[1] == d
-    n = out.shape[0]
-    assert n == (x.shape[0] if rows is None else rows.numel()) and weight.numel() == d
+    assert x.dtype == torch.float32 and x.is_contiguous() and (out is None or (out.is_contiguous() and out.shape[1] == d))
+    n = x.shape[0] if rows is None else rows.numel()
+    assert out is None or out.shape[0] == n
+    assert weight is None or weight.numel() == d
     w_post, post_eps, value = None, 0.0, delta
     if isinstance(delta, NormedDelta):
         w_post, post_eps, value = _f32(delta.weight, "weight"), delta.eps, delta.value
@@ -539,7 +550,7 @@ def sandwich_norm(x: torch.Tensor, delta, weight: torch.Tensor, eps: float, out:
     _check(lib().infero_sandwich_norm(
         _ptr(x), _ptr(y0), c_int(s0), c_longlong(st0), _ptr(b0), _ptr(_f32(w0, "w0")), _ptr(y1), c_int(s1), c_longlong(st1),
         _ptr(b1), _ptr(_f32(w1, "w1")), c_float(scale), c_float(branch_eps), _ptr(w_post), c_float(post_eps),
-        _ptr(_f32(weight, "weight")), c_float(eps), _ptr(out), c_int(_dt(out)),
+        _ptr(_f32(weight, "weight")), c_float(eps), _ptr(out), c_int(_dt(out) if out is not None else 0),
         _ptr(None if rows is None else _i32(rows, "rows")), c_int(n), c_int(d), _ptr(_f32(cw, "conv")), c_int(taps), _ptr(state),
         c_longlong(stride), _ptr(tok_entry), _ptr(entry_slot), _stream()))
 
@@ -560,10 +571,13 @@ def input_conv(h: torch.Tensor, w: torch.Tensor, state: torch.Tensor, tok_entry,
 
 # ---- embedding of a token, of its pair with the one before, and of its position (csrc/embed_compose.cu) -----------
 def embed_compose(table: torch.Tensor, ids: torch.Tensor, out_x: torch.Tensor, scale: float, device_tokens, bigram, previous,
-                  pos_table, positions, tok_entry, entry_q_start, entry_q_len, entry_slot, n_entries: int, single: bool) -> None:
+                  pos_table, positions, tok_entry, entry_q_start, entry_q_len, entry_slot, n_entries: int, single: bool,
+                  norm_w: Optional[torch.Tensor] = None, eps: float = 0.0, h: Optional[torch.Tensor] = None) -> None:
     """out_x[t] = table[id] * scale + bigram row + position row; ``bigram`` = (table, buckets, mul_prev, mul_cur) or None with
-    ``previous`` int32 [slots, 1] the last token of every request slot; ``single``: every request brings one token."""
+    ``previous`` int32 [slots, 1] the last token of every request slot; ``single``: every request brings one token.
+    ``norm_w`` float32 [d]: the sum is RMS-normed with that weight; ``h`` (bf16) receives a copy of the result."""
     T, d = out_x.shape
+    assert h is None or (h.dtype == torch.bfloat16 and h.is_contiguous() and h.shape == out_x.shape)
     assert out_x.dtype == torch.float32 and out_x.is_contiguous() and table.is_contiguous() and table.shape[1] == d
     bt, buckets, mp, mc = bigram if bigram is not None else (None, 0, 0, 0)
     assert bt is None or (bt.dtype == table.dtype and bt.is_contiguous() and tuple(bt.shape) == (buckets + 1, d))
@@ -574,11 +588,11 @@ def embed_compose(table: torch.Tensor, ids: torch.Tensor, out_x: torch.Tensor, s
         c_longlong(buckets), _ptr(None if previous is None else _i32(previous, "previous")), _ptr(_i32(tok_entry, "tok_entry")),
         _ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")),
         c_int(n_entries), _ptr(pos_table), c_int(pos_table.shape[0] if pos_table is not None else 0),
-        _ptr(_i32(positions, "positions")), c_int(1 if single else 0), _stream()))
+        _ptr(_i32(positions, "positions")), c_int(1 if single else 0), _ptr(_f32(norm_w, "norm_w")), c_float(eps), _ptr(h), _stream()))
 
 
 # ---- recurrences with a matrix per head (csrc/outer_memory.cu) -------------------------------------------------------
-MEMORY_RULES = {"delta": 0, "gated": 1}
+MEMORY_RULES = {"delta": 0, "gated": 1, "channel": 2, "decayed": 3}
 
 
 def memory_tail_floats(taps: int, channels: int) -> int:
@@ -638,7 +652,7 @@ def memory_gates(gates: torch.Tensor, in_off: int, forget_off: int, cap: float, 
 
 
 def _memory_scan(rule: str, src, q_off, k_off, v_off, table, gates, in_off, forget_off, cap, q_scale, state, s_off, entry_q_start,
-                 entry_q_len, entry_slot, n_entries, H, G, K, V, single):
+                 entry_q_len, entry_slot, n_entries, H, G, K, V, single, aux=None, group_decay=None):
     from .tc_gemm import sm_count
     T = src.shape[0]
     gated = rule == "gated"
@@ -653,7 +667,7 @@ def _memory_scan(rule: str, src, q_off, k_off, v_off, table, gates, in_off, forg
         c_float(q_scale), _ptr(state), c_longlong(state.stride(0)), c_longlong(s_off),
         _ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")),
         _ptr(y), _ptr(den), c_int(n_entries), c_int(1 if single else 0), c_int(H), c_int(G), c_int(K), c_int(V),
-        c_int(sm_count(src.device)), _stream()))
+        c_int(sm_count(src.device)), _ptr(aux), _ptr(group_decay), c_longlong(aux.stride(0) if aux is not None else 0), _stream()))
     return y, den
 
 
@@ -677,6 +691,68 @@ def gated_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, in_off: i
                              n_entries, H, V + 1)
     return _memory_scan("gated", proj, q_off, k_off, v_off, table, proj if single else None, in_off, forget_off, cap, K ** -0.5, state, s_off,
                         entry_q_start, entry_q_len, entry_slot, n_entries, H, H, K, V, single)
+
+
+# ---- memories with a decay per channel of a key (csrc/low_rank.cu, outer_memory_channel.cu, outer_memory_decayed.cu) -------
+LOW_RANK_MODES = {"plain": 0, "decay": 1, "sigmoid": 2}
+
+
+def low_rank(a: torch.Tensor, w: torch.Tensor, mode: str = "plain", bias: Optional[torch.Tensor] = None,
+             a_log: Optional[torch.Tensor] = None, tau: float = 1.0) -> torch.Tensor:
+    """float32 [T, N] from a product's narrow middle ``a`` (float32 [T, R], a column slice) and w [N, R]: z = a w^T (+ bias);
+    "decay": exp(-exp(a_log of the head) softplus(z)) with N / len(a_log) columns a head; "sigmoid": sigmoid(z)^(1 / tau)."""
+    T, R = a.shape
+    N = w.shape[0]
+    assert a.dtype == torch.float32 and a.stride(1) == 1 and w.is_contiguous() and w.shape[1] == R
+    assert bias is None or bias.numel() == N
+    assert mode != "decay" or N % a_log.numel() == 0
+    out = torch.empty((T, N), dtype=torch.float32, device=a.device)
+    _check(lib().infero_low_rank(_ptr(a), c_longlong(a.stride(0)), _ptr(w), c_int(_dt(w)), _ptr(_f32(bias, "bias")), _ptr(_f32(a_log, "a_log")),
+                                 c_int(N // a_log.numel() if a_log is not None else 1), c_float(tau), c_int(LOW_RANK_MODES[mode]), _ptr(out),
+                                 c_int(T), c_int(N), c_int(R), _stream()))
+    return out
+
+
+def channel_prepare(proj: torch.Tensor, x_off: int, step_off: int, conv_w: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
+                    tok_entry, entry_q_start, entry_q_len, entry_slot, n_entries: int, G: int, H: int, K: int, V: int, single: bool):
+    """What the delta rule's scan needs where every channel of a key decays on its own: (u [T, 4 H K + H V], table [H, T, 12])
+    from the 32-bit product rows ([q | k | v] at ``x_off``, raw steps at ``step_off``) and the decays [T, H K]; see
+    csrc/outer_memory_channel.cu.  The requests' tails (the convolution's last taps - 1 inputs) move on."""
+    T = proj.shape[0]
+    taps, CH = conv_w.shape
+    assert CH == 2 * G * K + H * V and proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= max(x_off + CH, step_off + H)
+    assert decay.dtype == torch.float32 and decay.is_contiguous() and tuple(decay.shape) == (T, H * K)
+    assert state.dtype == torch.float32 and state.is_contiguous()
+    u = torch.empty((T, 4 * H * K + H * V), dtype=torch.float32, device=proj.device)
+    table = torch.empty((H, T, 12), dtype=torch.float32, device=proj.device)
+    L = lib()
+    batch = (_ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")))
+    own_tail = single and H == G
+    _check(L.infero_channel_prepare(_ptr(proj), c_longlong(proj.stride(0)), c_int(x_off), _ptr(_f32(conv_w, "conv_w")), c_int(taps), _ptr(state),
+                                    c_longlong(state.stride(0)), _ptr(_i32(tok_entry, "tok_entry")), *batch, _ptr(u), _ptr(table), _ptr(decay),
+                                    c_int(step_off), c_int(T), c_int(G), c_int(H), c_int(K), c_int(V), c_int(1 if own_tail else 0), _stream()))
+    if not own_tail:
+        _check(L.infero_conv_tail(_ptr(proj[:, x_off:]), c_int(proj.stride(0)), c_int(taps), _ptr(state), c_longlong(state.stride(0)), *batch,
+                                  c_int(n_entries), c_int(CH), _stream()))
+    return u, table
+
+
+def channel_scan(u: torch.Tensor, table: torch.Tensor, state: torch.Tensor, s_off: int, entry_q_start, entry_q_len, entry_slot,
+                 n_entries: int, H: int, K: int, V: int, single: bool = False) -> torch.Tensor:
+    """The delta rule with a decay per channel, from what ``channel_prepare`` left; float32 [T, H V].  S [H, V, K] at ``s_off``."""
+    HK = H * K
+    assert table.is_contiguous() and tuple(table.shape) == (H, u.shape[0], 12) and u.shape[1] == 4 * HK + H * V
+    return _memory_scan("channel", u, 0, HK, 4 * HK, table, None, 0, 0, 0.0, 1.0, state, s_off, entry_q_start, entry_q_len, entry_slot,
+                        n_entries, H, H, K, V, single, aux=u[:, 2 * HK:], group_decay=u[:, 3 * HK:])[0]
+
+
+def decayed_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, state: torch.Tensor, s_off: int, entry_q_start,
+                 entry_q_len, entry_slot, n_entries: int, H: int, K: int, V: int, single: bool = False) -> torch.Tensor:
+    """Gated linear attention of every request over its new tokens, from the 32-bit product rows and the decays [T, H K];
+    float32 [T, H V], q times K^-1/2.  S [H, V, K] at ``s_off``."""
+    assert decay.dtype == torch.float32 and decay.is_contiguous() and tuple(decay.shape) == (proj.shape[0], H * K)
+    return _memory_scan("decayed", proj, q_off, k_off, v_off, None, None, 0, 0, 0.0, K ** -0.5, state, s_off, entry_q_start, entry_q_len,
+                        entry_slot, n_entries, H, H, K, V, single, aux=decay)[0]
 
 
 def memory_finish(y: torch.Tensor, den: Optional[torch.Tensor], gate: torch.Tensor, act: str, norm_w: torch.Tensor, eps: float,

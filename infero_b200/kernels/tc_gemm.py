@@ -81,14 +81,15 @@ def set_pairs(on: bool) -> None:
     lib().infero_gemm_set_pairs(c_int(1 if on else 0))
 
 
-def gemm_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
-    """out[M, N/2] = silu(g) * u where (g_j, u_j) are columns (2j, 2j+1) of a @ w^T.  Returns False
+def gemm_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None) -> bool:
+    """out[M, N/2] = silu(g) * u where (g_j, u_j) are columns (2j, 2j+1) of a @ w^T (+ bias).  Returns False
     (nothing launched) when few rows would need more than one split of K."""
     M, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.shape == (M, N // 2) and out.stride(1) == 1 and out.dtype == torch.bfloat16
-    rc = lib().infero_gemm_tc_swiglu(_ptr(a), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_int(a.stride(0)),
-                                     c_int(out.stride(0)), c_int(sm_count(a.device)), _stream())
+    assert bias is None or bias.numel() == N
+    rc = lib().infero_gemm_tc_swiglu_bias(_ptr(a), _ptr(w), _ptr(bias), c_int(_dt(bias) if bias is not None else F32), _ptr(out), c_int(M),
+                                          c_int(N), c_int(K), c_int(a.stride(0)), c_int(out.stride(0)), c_int(sm_count(a.device)), _stream())
     if rc == 2:
         return False
     _check(rc)

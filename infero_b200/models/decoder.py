@@ -27,6 +27,11 @@ class DecoderModel:
         self.spec = spec
         self.blocks = [part_class("block", b.kind)(b) for b in spec.blocks]
         self.final_norm = part_class("norm", spec.final_norm.kind)(spec.final_norm, spec.final_norm_name)
+        self.embed_norm = None
+        if spec.embed_norm is not None:
+            if spec.embed_norm.kind not in ("rmsnorm", "rmsnorm_centred"):
+                raise ValueError("the embedding takes an RMS norm")
+            self.embed_norm = part_class("norm", spec.embed_norm.kind)(spec.embed_norm, spec.embed_norm_name)
         self.embed: Optional[torch.Tensor] = None
         self.bigram: Optional[torch.Tensor] = None
         self.position_table: Optional[torch.Tensor] = None
@@ -77,6 +82,8 @@ class DecoderModel:
             out.append(TensorDecl(s.bigram.name, (s.bigram.buckets + 1, s.hidden), role="embedding"))
         if s.position_table:
             out.append(TensorDecl(s.position_table, (s.max_positions, s.hidden), role="embedding"))
+        if self.embed_norm is not None:
+            out += self.embed_norm.declare()
         for b in self.blocks:
             out += b.declare()
         out += self.final_norm.declare()
@@ -98,7 +105,13 @@ class DecoderModel:
             self.position_table = tensors[s.position_table].to(self.embed.dtype).contiguous()
         for b in self.blocks:
             b.bind(tensors)
+        if self.embed_norm is not None:
+            self.embed_norm.bind(tensors)
+            self.embed_norm.weight = self.embed_norm.weight.float().contiguous()
         self.final_norm.bind(tensors)
+        if s.logit_scale != 1.0:
+            # the logits' constant multiplies what the output product reads (its norm's weight, in 32-bit)
+            self.final_norm.weight = (self.final_norm.weight.float() * s.logit_scale).contiguous()
         # a tied head aliases the embedding (crates/model/src/weights.rs:2835-2849)
         self.head = Linear(self.embed if s.tie_embeddings else tensors[s.head_name], None, "lm_head")
 
@@ -151,10 +164,7 @@ class DecoderModel:
             total = torch.empty((R, s.hidden), dtype=torch.float32, device=x0.device)
             L.hyper_step(x, y, mix, w_out, None, None, 0.0, None, u_out=total, rows=logit_rows)
             h = self.final_norm.forward(ctx, total, None)
-        logits = self.head.forward(h, out_dtype=torch.float32)
-        if s.logit_scale != 1.0:
-            logits.mul_(s.logit_scale)
-        return logits
+        return self.head.forward(h, out_dtype=torch.float32)
 
     @property
     def position_limit(self) -> Optional[int]:
@@ -164,7 +174,7 @@ class DecoderModel:
     def _embed(self, ctx, token_ids: torch.Tensor, x: torch.Tensor) -> None:
         s = self.spec
         device_tokens = getattr(ctx, "device_tokens", None)
-        if s.bigram is None and not s.position_table:
+        if s.bigram is None and not s.position_table and self.embed_norm is None:
             K.embed_gather(self.embed, token_ids, x, s.embed_scale, device_tokens)
             return
         from ..kernels import layer_ops as L
@@ -172,8 +182,15 @@ class DecoderModel:
         if s.bigram is not None:
             big = (self.bigram, s.bigram.buckets, s.bigram.mul_prev, s.bigram.mul_cur)
             previous = ctx.state(self.MODEL, "previous_token")
+        norm_w, eps, h = None, 0.0, None
+        if self.embed_norm is not None:
+            norm_w, eps = self.embed_norm.weight, self.embed_norm.spec.eps
+        if ctx.act_dtype == torch.bfloat16 and not s.streams and s.blocks[s.schedule[0].block].kind == "postnorm":
+            h = torch.empty(x.shape, dtype=torch.bfloat16, device=x.device)     # the first block reads x itself
+            ctx._resid_act = (-1, h)
         L.embed_compose(self.embed, token_ids, x, s.embed_scale, device_tokens, big, previous, self.position_table, ctx.positions,
-                        ctx.tok_entry, ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, int(ctx.max_q_len) == 1)
+                        ctx.tok_entry, ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, int(ctx.max_q_len) == 1,
+                        norm_w=norm_w, eps=eps, h=h)
 
     # ---- one pass over the tokens of a step -------------------------------------------------
     def forward(self, ctx, token_ids: torch.Tensor, logit_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
@@ -204,7 +221,4 @@ class DecoderModel:
         if logit_rows is None or logit_rows.numel() == 0:
             return None
         h = self.final_norm.forward(ctx, x, delta, rows=logit_rows)
-        logits = self.head.forward(h, out_dtype=torch.float32)
-        if s.logit_scale != 1.0:
-            logits.mul_(s.logit_scale)
-        return logits
+        return self.head.forward(h, out_dtype=torch.float32)

@@ -51,7 +51,7 @@ class NativeDecoder:
         from ..parts.block import PreNormBlock
         from ..parts.norm import RmsNorm
         m = self.model
-        if m.spec.logit_scale != 1.0 or type(m.final_norm) is not RmsNorm or m.spec.bigram is not None or m.spec.position_table:
+        if m.spec.logit_scale != 1.0 or m.embed_norm is not None or type(m.final_norm) is not RmsNorm or m.spec.bigram is not None or m.spec.position_table:
             return False
         if not all(type(b) is PreNormBlock for b in m.blocks):
             return False

@@ -14,9 +14,9 @@ from .latent_attention import LatentAttention
 from .normed_attention import NormedAttention
 from .rglru import RgLruMixer
 from .ssd import SsdMixer
-from .outer_memory import DeltaMemory, GatedMemory
+from .outer_memory import ChannelDeltaMemory, DecayedMemory, DeltaMemory, GatedMemory
 from .parallel import ParallelMixer
-from .block import GatedPostNormBlock, HyperPreNormBlock, PreNormBlock, SandwichBlock
+from .block import GatedPostNormBlock, HyperPreNormBlock, PostNormBlock, PreNormBlock, SandwichBlock
 
 register_part("norm", "rmsnorm", RmsNorm)
 register_part("position", "rope_neox", RopeNeox)
@@ -44,9 +44,12 @@ register_part("norm", "rmsnorm_centred", CentredRmsNorm)
 register_part("mixer", "delta_memory", DeltaMemory)
 register_part("mixer", "gated_memory", GatedMemory)
 register_part("block", "sandwich", SandwichBlock)
+register_part("block", "postnorm", PostNormBlock)
+register_part("mixer", "channel_delta_memory", ChannelDeltaMemory)
+register_part("mixer", "decayed_memory", DecayedMemory)
 
 __all__ = ["FeedForward", "KvCacheSpec", "Mixer", "Norm", "Part", "PositionEncoding", "StateSpec",
            "TensorDecl", "Linear", "RmsNorm", "ScalarRmsNorm", "RopeNeox", "RopeInterleaved", "SwiGluMlp", "GqaAttention",
            "Hgrn2Mixer", "DiffAttention", "MoeSwiGlu", "PreNormBlock", "GatedPostNormBlock", "LayerNorm", "GluMlp", "Relu2Mlp",
            "GroupedMoe", "LatentAttention", "HyperPreNormBlock", "NormedAttention", "RgLruMixer", "ParallelMixer", "SsdMixer", "ScoredMoe",
-           "CentredRmsNorm", "DeltaMemory", "GatedMemory", "SandwichBlock"]
+           "CentredRmsNorm", "DeltaMemory", "GatedMemory", "SandwichBlock", "PostNormBlock", "ChannelDeltaMemory", "DecayedMemory"]

@@ -165,6 +165,80 @@ class SandwichBlock(Part):
         return K.NormedDelta(self.ffn.forward(ctx, h), self.ffn_post.weight, self.ffn_post.spec.eps)
 
 
+class PostNormBlock(Part):
+    """The sublayers read the residual stream itself, and a norm sits on their results only:
+
+        x += norm1(mixer(x));   x += norm2(ffn(x))
+
+    with RMS norms.  A sublayer's result stays pending as a ``NormedDelta``: the kernel in front of the next sublayer norms it,
+    adds it to x (32-bit) and leaves the new x in the step's element type for the sublayer's products, in one pass.  In
+    32-bit the sublayers read x where it is."""
+
+    def __init__(self, spec: BlockSpec):
+        self.spec = spec
+        p = spec.prefix
+        norm = lambda s, leaf: part_class("norm", s.kind)(s, f"{p}.{leaf}")      # noqa: E731
+        self.mixer_norm = norm(spec.mixer_norm, spec.mixer_norm_name)
+        self.mixer = part_class("mixer", spec.mixer.kind)(spec.mixer, p)
+        self.ffn = self.ffn_norm = None
+        if spec.ffn is not None:
+            self.ffn_norm = norm(spec.ffn_norm, spec.ffn_norm_name)
+            self.ffn = part_class("feed_forward", spec.ffn.kind)(spec.ffn, p)
+        if any(n.spec.kind not in ("rmsnorm", "rmsnorm_centred") for n in (self.mixer_norm, self.ffn_norm) if n is not None):
+            raise ValueError("a post-norm block takes RMS norms")
+
+    def parts(self):
+        return [p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None]
+
+    def declare(self) -> List[TensorDecl]:
+        out: List[TensorDecl] = []
+        for part in self.parts():
+            out += part.declare()
+        return out
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        for part in self.parts():
+            part.bind(tensors)
+        for n in (self.mixer_norm, self.ffn_norm):
+            if n is not None:
+                n.weight = n.weight.float().contiguous()
+
+    @staticmethod
+    def _advance(ctx, x, delta):
+        """x with what is pending added, and what the next sublayer reads."""
+        from .. import kernels as K
+        from ..kernels import layer_ops as L
+        if hasattr(delta, "as_partials"):
+            delta = delta.as_partials()
+        if isinstance(delta, K.Scaled) or (isinstance(delta, torch.Tensor) and delta.dtype != torch.float32):
+            # left pending by a block of another kind
+            scale = delta.scale if isinstance(delta, K.Scaled) else 1.0
+            value = delta.value if isinstance(delta, K.Scaled) else delta
+            if isinstance(value, K.Partials):
+                value = value.materialize(torch.float32)
+            K.residual_add(x, (value.float() * scale).contiguous())
+            delta = None
+        if ctx.act_dtype == torch.float32:
+            if delta is not None:
+                L.sandwich_norm(x, delta, None, 0.0, None)
+            return x
+        left = getattr(ctx, "_resid_act", None)
+        if delta is None and left is not None and left[0] == getattr(ctx, "schedule_index", -2) - 1 and left[1].shape == x.shape:
+            return left[1]                   # the embedding's own kernel left it
+        h = torch.empty(x.shape, dtype=ctx.act_dtype, device=x.device)
+        L.sandwich_norm(x, delta, None, 0.0, h)
+        return h
+
+    def forward(self, ctx, x, delta, slot):
+        from .. import kernels as K
+        h = self._advance(ctx, x, delta)
+        y = K.NormedDelta(self.mixer.forward(ctx, h, slot), self.mixer_norm.weight, self.mixer_norm.spec.eps)
+        if self.ffn is None:
+            return y
+        h = self._advance(ctx, x, y)
+        return K.NormedDelta(self.ffn.forward(ctx, h), self.ffn_norm.weight, self.ffn_norm.spec.eps)
+
+
 class GatedPostNormBlock(Part):
     """The sublayers read the residual stream itself; the norm sits on their result, behind a gate:
 

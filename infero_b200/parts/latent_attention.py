@@ -29,7 +29,9 @@ class LatentAttention(Mixer):
     be 0 (no rotated part: positions enter through the causal mask alone).
 
     ``q_latent_dim`` = Q > 0: the queries have a latent of their own.  The stacked product gives [dq | down (| gate)], the
-    first Q columns are RMS-normed with a weight (32-bit) and a second product with Wuq [H (D + R), Q] gives the queries."""
+    first Q columns are RMS-normed with a weight (32-bit) and a second product with Wuq [H (D + R), Q] gives the queries.
+
+    ``window``: a token sees that many keys up to its own; ``sink_per_head``: a learned sink in every head's softmax."""
 
     def __init__(self, spec: MixerSpec, prefix: str):
         self.spec, self.prefix = spec, prefix
@@ -37,8 +39,6 @@ class LatentAttention(Mixer):
         self.Q = int(spec.q_latent_dim)
         if min(self.H, self.D, self.V, self.C) <= 0 or self.R < 0 or self.Q < 0:
             raise ValueError("latent attention needs heads, head_dim, value_dim and latent_dim")
-        if spec.window:
-            raise ValueError("latent attention keeps every key")
         self.names = spec.tensor_names()
         self.rope, self.pairing, self.amp = None, "half", 1.0
         if spec.position is not None and spec.position.rotary_dim > 0:
@@ -54,10 +54,10 @@ class LatentAttention(Mixer):
 
     def _n(self, role: str) -> str:
         leaf = self.names[role]
-        return f"{self.prefix}.{leaf}" + ("" if role in ("latent_norm", "q_norm") else self.spec.weight_suffix)
+        return f"{self.prefix}.{leaf}" + ("" if role in ("latent_norm", "q_norm", "sink") else self.spec.weight_suffix)
 
     def cache_spec(self) -> Optional[KvCacheSpec]:
-        return KvCacheSpec(1, self.C + self.R, None, v_head_dim=0)        # the values are the first C columns of a key row
+        return KvCacheSpec(1, self.C + self.R, self.spec.window, v_head_dim=0)        # the values are the first C columns of a key row
 
     def declare(self) -> List[TensorDecl]:
         d, H, D, R, V, C = self.spec.hidden, self.H, self.D, self.R, self.V, self.C
@@ -72,6 +72,8 @@ class LatentAttention(Mixer):
                TensorDecl(self._n("o"), (d, H * V))]
         if self.spec.out_gate:
             out.append(TensorDecl(self._n("gate"), (H, d)))
+        if self.spec.sink_per_head:
+            out.append(TensorDecl(self._n("sink"), (H,), role="bias"))
         return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -89,6 +91,10 @@ class LatentAttention(Mixer):
             self.q_norm = tensors[self._n("q_norm")].float().contiguous()
             self.q_up = Linear(tensors[self._n("q_up")], None, self._n("q_up"))
         self.latent_norm = tensors[self._n("latent_norm")].float().contiguous()
+        self.sinks = self.sinks_log2 = None
+        if self.spec.sink_per_head:
+            self.sinks = tensors[self._n("sink")].float().contiguous()
+            self.sinks_log2 = (self.sinks * 1.4426950408889634).contiguous()
         # [H, C, D]: head n's rows of Wuk, transposed, so that the product with the plain query parts is a @ w^T
         self.up_k_t = tensors[self._n("up_k")].view(H, D, C).transpose(1, 2).contiguous()
         self.up_v = tensors[self._n("up_v")].view(H, V, C).contiguous()
@@ -118,7 +124,7 @@ class LatentAttention(Mixer):
         q_lat = torch.empty((H, rows, C), dtype=torch.float32, device=dev)
         A.per_head_product(q_plain, self.up_k_t, q_lat, T)
         o_lat = torch.empty((H, rows, C), dtype=h.dtype, device=dev)
-        A.attention(ctx, q_lat, q_rot, o_lat, kv, table, T, H, C, R, self.spec.scale)
+        A.attention(ctx, q_lat, q_rot, o_lat, kv, table, T, H, C, R, self.spec.scale, self.spec.window, self.sinks, self.sinks_log2)
         val = torch.empty((H, rows, V), dtype=torch.float32, device=dev)
         A.per_head_product(o_lat, self.up_v, val, T)
         attn = torch.empty((T, H * V), dtype=h.dtype, device=dev)

@@ -18,7 +18,8 @@ class SwiGluMlp(FeedForward):
     side by side: the tensor-core kernel applies the activation in its epilogue, and where it
     cannot (32-bit path, a product cut into several splits) the SwiGLU kernel takes the same
     alternating layout.  Where the tensors live under the block's prefix is data of the spec
-    (``FeedForwardSpec.names``): separate gate and up, or one stored [gate; up] tensor."""
+    (``FeedForwardSpec.names``): separate gate and up, or one stored [gate; up] tensor.  ``bias``: every projection has
+    one (leaf name + ``.b``), added in the products' epilogues or by the kernel that adds up partial sums."""
 
     def __init__(self, spec: FeedForwardSpec, prefix: str):
         self.spec = spec
@@ -31,12 +32,18 @@ class SwiGluMlp(FeedForward):
     def _n(self, role: str) -> str:
         return f"{self.prefix}.{self.names[role]}{self.spec.weight_suffix}"
 
+    def _b(self, role: str) -> str:
+        return f"{self.prefix}.{self.names[role]}.b"
+
     def declare(self) -> List[TensorDecl]:
         d, ff = self.spec.hidden, self.spec.intermediate
+        biases = [TensorDecl(self._b(r), (n,), role="bias") for r, n in (("gate", ff), ("up", ff), ("down", d))] if self.spec.bias else []
         if self.stored_stacked:
+            if biases:
+                raise ValueError("biases come with separate gate and up tensors")
             return [TensorDecl(self._n("gate_up"), (2 * ff, d)), TensorDecl(self._n("down"), (d, ff))]
         return [TensorDecl(self._n("gate"), (ff, d)), TensorDecl(self._n("up"), (ff, d)),
-                TensorDecl(self._n("down"), (d, ff))]
+                TensorDecl(self._n("down"), (d, ff))] + biases
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         if self.stored_stacked:
@@ -45,14 +52,22 @@ class SwiGluMlp(FeedForward):
             g, u = tensors[self._n("gate")], tensors[self._n("up")]
         if g.dtype != u.dtype:
             g, u = g.float(), u.float()
-        self.gate_up = Linear(torch.stack([g, u], dim=1).reshape(2 * g.shape[0], g.shape[1]), None,
+        gu_bias = down_bias = None
+        if self.spec.bias:
+            gu_bias = torch.stack([tensors[self._b("gate")].float(), tensors[self._b("up")].float()], dim=1).reshape(-1).contiguous()
+            down_bias = tensors[self._b("down")].float().contiguous()
+        self.gate_up = Linear(torch.stack([g, u], dim=1).reshape(2 * g.shape[0], g.shape[1]), gu_bias,
                               f"{self.prefix}.gate_up")
-        self.down = Linear(tensors[self._n("down")], None, self._n("down"))
+        self.down = Linear(tensors[self._n("down")], down_bias, self._n("down"))
 
     def forward(self, ctx, h):
         T = h.shape[0]
         act = torch.empty((T, self.spec.intermediate), dtype=h.dtype, device=h.device)
         if not self.gate_up.forward_swiglu(h, act):
+            if self.spec.bias:
+                from ..kernels import layer_ops as L
+                L.glu_act(self.gate_up.forward(h, defer=True, out_dtype=torch.float32), act)
+                return self.down.forward(act, defer=True, residual=True)
             K.swiglu(self.gate_up.forward(h, defer=True), act)
         return self.down.forward(act, defer=True, residual=True)
 
@@ -66,6 +81,8 @@ class GluMlp(SwiGluMlp):
         s = self.spec
         if s.activation == "swiglu":
             return super().forward(ctx, h)
+        if s.bias:
+            raise ValueError("the clamped activation comes without biases")
         from ..kernels import layer_ops as L, tc_gemm
         act = torch.empty((h.shape[0], s.intermediate), dtype=h.dtype, device=h.device)
         # many rows in bf16: the activation in the product's epilogue; else the product (as partial sums where it is cut)

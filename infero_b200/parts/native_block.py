@@ -131,7 +131,7 @@ class NativeBlock:
         from .norm import RmsNorm
         from .rope import RopeNeox
         b = self.block
-        if type(b.mixer) is not GqaAttention or type(b.ffn) is not SwiGluMlp:
+        if type(b.mixer) is not GqaAttention or type(b.ffn) is not SwiGluMlp or b.ffn.spec.bias:
             return False
         if float(getattr(b.spec, "residual_scale", 1.0)) != 1.0:
             return False

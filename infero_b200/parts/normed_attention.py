@@ -48,7 +48,8 @@ class NormedAttention(Mixer):
     by the heads, before the rotation) and appends keys and values to the cache; then attention (causal, optionally
     windowed, optionally with a sink in the softmax's denominator, optionally with a distance bias: head h's score
     loses 2^(-b (h + 1) / H) times the distance to the key, b = ``distance_slope_exp``; optionally with a learned bias by
-    distance and head, ``distance_buckets``), an optional sigmoid gate per head or (``gate_per_channel``) per number, and the
+    distance and head, ``distance_buckets``; optionally with a learned sink per head, ``sink_per_head``, and a soft cap of the
+    scaled scores, ``softcap``), an optional sigmoid gate per head or (``gate_per_channel``) per number, and the
     output product (with a bias where ``out_bias`` says so).
 
     ``head_mix``: the heads' softmax weights are mixed by a stored [H, H] matrix before they meet the values.  Attention
@@ -90,6 +91,12 @@ class NormedAttention(Mixer):
         self.n_rows = self.g_off + self.n_gates
         if spec.head_mix and (spec.sink or spec.distance_slope_exp > 0):
             raise ValueError("mixed heads come without a sink and without slopes")
+        if spec.head_mix and (spec.sink_per_head or spec.softcap > 0):
+            raise ValueError("mixed heads come without learned sinks and without a soft cap")
+        if spec.sink and spec.sink_per_head:
+            raise ValueError("one kind of sink")
+        if spec.scale_values and not (self.own_v and not spec.out_gate and not spec.head_mix):
+            raise ValueError("only ungated values of a projection of their own can carry the branch's scale")
         if spec.head_mix and spec.out_gate and not spec.gate_per_channel:
             raise ValueError("mixed heads are gated per channel")
         self.inp: Linear = None
@@ -127,6 +134,8 @@ class NormedAttention(Mixer):
             out.append(TensorDecl(self._n("o_bias", False), (d,), role="bias"))
         if s.distance_buckets:
             out.append(TensorDecl(self._n("distance", False), (s.distance_buckets, self.H), role="bias", free_axes=(0,)))
+        if s.sink_per_head:
+            out.append(TensorDecl(self._n("sink", False), (self.H,), role="bias"))
         if s.head_mix:
             out.append(TensorDecl(self._n("head_mix", False), (self.H, self.H), role="bias", init="eye"))
         return out
@@ -148,7 +157,10 @@ class NormedAttention(Mixer):
         self.inp = Linear(self._rows, self._bias, f"{self.prefix}.qkv")
         self._out_w = tensors[self._n("o")]
         self.out = Linear(self._out_w, tensors[self._n("o_bias", False)].float().contiguous() if s.out_bias else None, self._n("o"))
-        self.rel = self.rel_log2 = self.mix = None
+        self.rel = self.rel_log2 = self.mix = self.sinks = self.sinks_log2 = None
+        if s.sink_per_head:
+            self.sinks = tensors[self._n("sink", False)].float().contiguous()
+            self.sinks_log2 = (self.sinks * 1.4426950408889634).contiguous()
         if s.distance_buckets:
             # the table by distance, [H, distances]: the last entry stands for every distance from there on
             table = tensors[self._n("distance", False)].float()
@@ -193,9 +205,13 @@ class NormedAttention(Mixer):
         freq = self.rope.inv_freq64(dev) if self.rope is not None else None
         amp = float(getattr(self.rope, "amplitude", 1.0)) if self.rope is not None else 1.0
         q = torch.empty((T, H * D), dtype=ctx.act_dtype, device=dev)
+        v_scale = 1.0
+        if s.scale_values:                     # attention is linear in the values: they are cached times the scale
+            v_scale, scale = scale, 1.0
         L.qk_prepare(proj, off + self.q_off, off + self.k_off if self.own_kv else -1, off + self.v_off if self.own_v else -1,
                      self.NORM_MODES[s.qk_norm_kind], self.q_norm, self.k_norm, s.norm_eps, freq, amp, ctx.positions,
-                     ctx.tok_entry, table, kv.page_size, q, kv.k, kv.v, H, G, D, V, write_cache=write)
+                     ctx.tok_entry, table, kv.page_size, q, kv.k, kv.v, H, G, D, V, write_cache=write,
+                     temperature=s.q_temperature, v_scale=v_scale)
         gate = proj[:, off + self.g_off:off + self.g_off + self.n_gates] if s.out_gate else None
         if s.head_mix:
             from ..kernels import attention as A
@@ -205,7 +221,8 @@ class NormedAttention(Mixer):
         direct = not s.out_gate and scale == 1.0
         attn = out if direct else torch.empty((T, H * V), dtype=ctx.act_dtype, device=dev)
         from ..kernels import attention as A
-        A.paged_attention_ex(ctx, q, attn, kv, table, H, G, D, V, s.window, s.scale, s.sink, slopes=self.slopes, rel=self.rel)
+        A.paged_attention_ex(ctx, q, attn, kv, table, H, G, D, V, s.window, s.scale, s.sink, slopes=self.slopes, rel=self.rel,
+                             rel_log2=self.rel_log2, sinks=self.sinks, sinks_log2=self.sinks_log2, softcap=float(s.softcap))
         if not direct:
             per_head = not s.gate_per_channel
             L.head_gate(attn, gate, out, H if per_head else H * V, V if per_head else 1, scale)

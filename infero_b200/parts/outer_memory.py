@@ -169,3 +169,140 @@ class GatedMemory(_OuterMemory):
                               single_tokens(ctx))
         L.memory_finish(y, den, proj[:, off + o["gate"]:off + o["gate"] + H * V], "sigmoid", self.norm_w, float(self.spec.norm_eps),
                         out, H, V, scale)
+
+
+class _ChannelDecayed(_OuterMemory):
+    """Memories whose every key channel decays on its own.  The decays (and a gate, where the rule has one of that kind) are
+    products through a narrow middle, W_up (W_down h): the rows of W_down ride on the stacked input product and ``low_rank``
+    does the rest in 32-bit.  How wide a middle is only the stored tensors say (``spec.low_rank`` where weights are made)."""
+
+    NARROW: Tuple[str, ...] = ()             # roles of the W_down
+
+    def __init__(self, spec: MixerSpec, prefix: str):
+        super().__init__(spec, prefix)
+        self.ranks = {r: int(spec.low_rank) for r in self.NARROW}
+        if min(self.ranks.values()) <= 0:
+            raise ValueError("a product through a narrow middle needs low_rank")
+        self.off = self._offsets()
+
+    def _declare_rows(self) -> List[TensorDecl]:
+        d = self.spec.hidden
+        return [TensorDecl(self._n(r), (n, d), free_axes=(0,) if r in self.NARROW else ()) for r, n in self._stack()]
+
+    def _bind_rows(self, tensors) -> None:
+        """The stacked product, its width rounded up to whole vectors of four."""
+        self.ranks = {r: tensors[self._n(r)].shape[0] for r in self.NARROW}
+        self.off = self._offsets()
+        self._bind_product(tensors)
+        pad = -self.n_rows % 4
+        if pad:
+            self._rows = torch.cat([self._rows, torch.zeros((pad, self._rows.shape[1]), dtype=self._rows.dtype, device=self._rows.device)])
+            self.inp = Linear(self._rows, None, self.inp.name)
+
+    def _up(self, tensors, role: str, down: str) -> torch.Tensor:
+        w = tensors[self._n(role)].contiguous()
+        if w.shape[1] != self.ranks[down]:
+            raise ValueError(f"{self._n(role)} takes {w.shape[1]} numbers, {self._n(down)} gives {self.ranks[down]}")
+        return w
+
+    def _narrow(self, proj: torch.Tensor, off: int, role: str) -> torch.Tensor:
+        at = off + self.off[role]
+        return proj[:, at:at + self.ranks[role]]
+
+
+class ChannelDeltaMemory(_ChannelDecayed):
+    """The gated delta rule with a decay per key channel.  One input product gives [q | k | v | decay's middle | gate's middle |
+    step]; ``low_rank`` makes the decays exp(-exp(A_log) softplus(W_a2 (W_a1 h) + dt_bias)) and the gate, then
+    ``channel_prepare`` (convolution, silu, unit vectors, what the scan reads of every group of four tokens) -> ``channel_scan``
+    -> ``memory_finish`` (RMS norm with a weight shared by the heads, sigmoid gate) -> output product.  The request's state: the
+    convolution's last taps - 1 inputs, then S."""
+
+    RULE = "channel_delta"
+    NARROW = ("decay_down", "gate_down")
+
+    def __init__(self, spec: MixerSpec, prefix: str):
+        self.G, self.taps = int(spec.num_kv_heads) or int(spec.num_heads), int(spec.conv_taps)
+        super().__init__(spec, prefix)
+        if self.H % self.G:
+            raise ValueError(f"{self.H} heads are not a multiple of {self.G} kv heads")
+        if not 1 <= self.taps <= 16:
+            raise ValueError(f"{self.taps} taps outside 1..16")
+        self.CH = 2 * self.G * self.K + self.H * self.V
+        self.s_off = L.memory_tail_floats(self.taps, self.CH)
+
+    def _stack(self):
+        return [("q", self.G * self.K), ("k", self.G * self.K), ("v", self.H * self.V), ("decay_down", self.ranks["decay_down"]),
+                ("gate_down", self.ranks["gate_down"]), ("step", self.H)]
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec((L.memory_state_floats("channel", self.H, self.K, self.V, self.taps, self.CH),), torch.float32)
+
+    def declare(self) -> List[TensorDecl]:
+        d, r = self.spec.hidden, self.ranks
+        out = self._declare_rows()
+        out += [TensorDecl(self._n(n + "_conv", False), (w, self.taps), role="bias", init="conv") for n, w in self._stack()[:3]]
+        return out + [TensorDecl(self._n("decay_up"), (self.H * self.K, r["decay_down"]), free_axes=(1,)),
+                      TensorDecl(self._n("gate_up"), (self.H * self.V, r["gate_down"]), free_axes=(1,)),
+                      TensorDecl(self._n("dt_bias", False), (self.H * self.K,), role="bias"), TensorDecl(self._n("a_log", False), (self.H,), role="bias"),
+                      TensorDecl(self._n("out_norm", False), (self.V,), role="norm", init="ones"),
+                      TensorDecl(self._n("o"), (d, self.H * self.V))]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        f32 = lambda r: tensors[self._n(r, False)].float().contiguous()          # noqa: E731
+        self._bind_rows(tensors)
+        self.decay_up, self.gate_up = self._up(tensors, "decay_up", "decay_down"), self._up(tensors, "gate_up", "gate_down")
+        self.conv_w = torch.cat([f32(r + "_conv") for r in ("q", "k", "v")], dim=0).t().contiguous()      # [taps, channels]
+        self.dt_bias, self.a_log, self.norm_w = f32("dt_bias"), f32("a_log"), f32("out_norm")
+
+    def core(self, ctx, proj: torch.Tensor, off: int, slot, out: torch.Tensor, scale: float = 1.0) -> None:
+        H, G, K, V = self.H, self.G, self.K, self.V
+        state, single = ctx.state(slot.cache), single_tokens(ctx)
+        decay = L.low_rank(self._narrow(proj, off, "decay_down"), self.decay_up, "decay", self.dt_bias, self.a_log)
+        gate = L.low_rank(self._narrow(proj, off, "gate_down"), self.gate_up)
+        batch = (ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries)
+        u, table = L.channel_prepare(proj, off, off + self.off["step"], self.conv_w, decay, state, ctx.tok_entry, *batch, G, H, K, V, single)
+        y = L.channel_scan(u, table, state, self.s_off, *batch, H, K, V, single)
+        L.memory_finish(y, None, gate, "sigmoid", self.norm_w, float(self.spec.norm_eps), out, H, V, scale)
+
+
+class DecayedMemory(_ChannelDecayed):
+    """Gated linear attention: S <- diag(a) S + k v^T, o = S^T q, with decays a = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau) per key
+    channel and every head its own q and k.  One input product gives [q | k | v | gate | decay's middle]; ``low_rank`` (decays)
+    -> ``decayed_scan`` -> ``memory_finish`` (RMS norm with a weight shared by the heads, silu gate) -> output product.  The
+    request's state: S."""
+
+    RULE = "decayed"
+    NARROW = ("decay_down",)
+
+    def __init__(self, spec: MixerSpec, prefix: str):
+        super().__init__(spec, prefix)
+        if not spec.decay_tau > 0:
+            raise ValueError("gated linear attention needs decay_tau")
+
+    def _stack(self):
+        return [("q", self.H * self.K), ("k", self.H * self.K), ("v", self.H * self.V), ("gate", self.H * self.V),
+                ("decay_down", self.ranks["decay_down"])]
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec((L.memory_state_floats("decayed", self.H, self.K, self.V),), torch.float32)
+
+    def declare(self) -> List[TensorDecl]:
+        return self._declare_rows() + [
+            TensorDecl(self._n("decay_up"), (self.H * self.K, self.ranks["decay_down"]), free_axes=(1,)),
+            TensorDecl(self._n("decay_bias", False), (self.H * self.K,), role="bias"),
+            TensorDecl(self._n("out_norm", False), (self.V,), role="norm", init="ones"),
+            TensorDecl(self._n("o"), (self.spec.hidden, self.H * self.V))]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        f32 = lambda r: tensors[self._n(r, False)].float().contiguous()          # noqa: E731
+        self._bind_rows(tensors)
+        self.decay_up = self._up(tensors, "decay_up", "decay_down")
+        self.decay_bias, self.norm_w = f32("decay_bias"), f32("out_norm")
+
+    def core(self, ctx, proj: torch.Tensor, off: int, slot, out: torch.Tensor, scale: float = 1.0) -> None:
+        H, K, V, o = self.H, self.K, self.V, self.off
+        decay = L.low_rank(self._narrow(proj, off, "decay_down"), self.decay_up, "sigmoid", self.decay_bias, tau=float(self.spec.decay_tau))
+        y = L.decayed_scan(proj, off + o["q"], off + o["k"], off + o["v"], decay, ctx.state(slot.cache), 0, ctx.entry_q_start, ctx.entry_q_len,
+                           ctx.entry_slot, ctx.n_entries, H, K, V, single_tokens(ctx))
+        L.memory_finish(y, None, proj[:, off + o["gate"]:off + o["gate"] + H * V], "silu", self.norm_w, float(self.spec.norm_eps), out,
+                        H, V, scale)

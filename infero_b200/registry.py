@@ -99,6 +99,8 @@ def _register_builtin() -> None:
     register_architecture("Pibavik", PibavikConfig.from_dict, lambda c: c.to_model_spec())
     from .config.nuvarax import NuvaraxConfig
     register_architecture("Nuvarax", NuvaraxConfig.from_dict, lambda c: c.to_model_spec())
+    from .config.dukolorn import DukolornConfig
+    register_architecture("Dukolorn", DukolornConfig.from_dict, lambda c: c.to_model_spec())
 
 
 _register_builtin()
