@@ -287,7 +287,7 @@ def main(argv=None) -> int:
                     help="instead of the headline workload: one of the added designs (--design) beside Qwen2 at equal layer sizes, prompt and decode "
                          "steps and the kernels alone (infero_b200/tools/design_bench.py; its own JSON line)")
     ap.add_argument("--design-sizes", default="s,m")
-    ap.add_argument("--design", default="vufizen", choices=["vufizen", "gositar", "banelix", "pibavik", "nuvarax"],
+    ap.add_argument("--design", default="vufizen", choices=["vufizen", "gositar", "banelix", "pibavik", "nuvarax", "dukolorn"],
                     help="with --designs: which of the added designs runs beside Qwen2 (pibavik: beside Banelix; nuvarax: beside Pibavik "
                          "and Banelix, the closest designs)")
     args = ap.parse_args(argv)

@@ -1,7 +1,7 @@
-"""Vufizen, Gositar or Banelix beside Qwen2, Pibavik beside Banelix, or Nuvarax beside Pibavik and Banelix, at equal layer sizes:
-whole prompt steps and decode steps, and the designs' own kernels one by one against their rooflines.
+"""Vufizen, Gositar or Banelix beside Qwen2, Pibavik beside Banelix, Nuvarax beside Pibavik and Banelix, or Dukolorn beside Nuvarax, at
+equal layer sizes: whole prompt steps and decode steps, and the designs' own kernels one by one against their rooflines.
 
-    python -m infero_b200.tools.design_bench [--design vufizen|gositar|banelix|pibavik|nuvarax] [--sizes s,m] [--prompt 2048]
+    python -m infero_b200.tools.design_bench [--design vufizen|gositar|banelix|pibavik|nuvarax|dukolorn] [--sizes s,m] [--prompt 2048]
                                              [--context 2048] [--batch 8] [--layers 8]
 
 (also ``bench.py --designs``).  Random weights made on the device, bf16.  Per size two models of the same width
@@ -28,6 +28,11 @@ Nuvarax (``--design nuvarax``): delta-rule layers and parallel layers (attention
 beside a gated matrix memory) alternating, a dense clamped gated feed-forward, norms before and after every sublayer and a
 convolution on what every mixer reads; beside Pibavik (the closest mixers: biased attention, a recurrence with a matrix per
 head) and Banelix (parallel layers with a dense feed-forward) of the same width, depth and (active) feed-forward width.
+
+Dukolorn (``--design dukolorn``): of every four layers one delta-rule layer with decays per channel, two parallel layers (soft-capped
+attention with a distance bias and learned sinks beside gated linear attention) and one latent attention layer over a window,
+a dense SwiGLU with biases and a norm on every sublayer's result; beside Nuvarax (delta-rule memories, biased attention beside a
+gated matrix memory) of the same width, depth, head counts, memory sizes and feed-forward.
 """
 from __future__ import annotations
 
@@ -108,6 +113,28 @@ NUVARAX_SIZES = {
     "l": dict(width=4096, heads=16, kv=4, dim=128, bias_max=512, mem_heads=32, mem_dim=128, mem_vdim=128, delta_heads=32,
               delta_kv=16, delta_dim=128, delta_vdim=128, taps=4, ff=11008, vocab=32000, beside="l"),
 }
+
+
+DUKOLORN_SIZES = {
+    "t": dict(NUVARAX_SIZES["t"], lat_heads=4, lat_dim=32, lat_rot=16, lat_vdim=32, lat_rank=64, window=48),      # for tests
+    "s": dict(NUVARAX_SIZES["s"], lat_heads=8, lat_dim=64, lat_rot=32, lat_vdim=64, lat_rank=256, window=1024),
+    "m": dict(NUVARAX_SIZES["m"], lat_heads=16, lat_dim=128, lat_rot=64, lat_vdim=128, lat_rank=512, window=1024),
+    "l": dict(NUVARAX_SIZES["l"], lat_heads=32, lat_dim=128, lat_rot=64, lat_vdim=128, lat_rank=512, window=1024),
+}
+
+
+def dukolorn_config(z, layers):
+    D = z["dim"]
+    delta = {"heads": z["delta_heads"], "kv_heads": z["delta_kv"], "dim": z["delta_dim"], "vdim": z["delta_vdim"], "conv": z["taps"]}
+    left = {"heads": z["heads"], "kv_heads": z["kv"], "dim": D, "vdim": D, "scale": D ** -0.5, "bias_max": z["bias_max"], "softcap": 30.0,
+            "q_temp": {"coef": 0.1, "every": 1024}}
+    par = {"left": left, "right": {"heads": z["mem_heads"], "dim": z["mem_dim"], "vdim": z["mem_vdim"], "tau": 16.0}, "left_scale": 0.9,
+           "right_scale": 1.1}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["lat_rot"], "vdim": z["lat_vdim"], "kv_rank": z["lat_rank"],
+           "scale": (z["lat_dim"] + z["lat_rot"]) ** -0.5, "rot": {"base": 10000.0, "dims": z["lat_rot"]}, "mask": {"size": z["window"]}}
+    kinds = [("channel_delta", delta), ("parallel", par), ("latent_attention", lat), ("parallel", par)]
+    return {"architecture": "Dukolorn", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "layers": [{"type": k, "mixer": m, "mlp": {"kind": "dense", "ff": z["ff"]}} for k, m in (kinds[i % 4] for i in range(layers))]}
 
 
 def nuvarax_config(z, layers, max_positions=4096):
@@ -909,9 +936,170 @@ def time_nuvarax_kernels(z, T, context, batch, timer, peaks):
     return rows
 
 
+def time_dukolorn_kernels(z, T, context, batch, timer, peaks):
+    """Dukolorn's kernels alone, each beside the kernel of another design that does the like job."""
+    import numpy as np
+    import torch
+    from infero_b200 import kernels as K
+    from infero_b200.kernels import attention as A, latent_attention as LA, layer_ops as L
+    from infero_b200.parts.linear import Linear
+    from infero_b200.parts.normed_attention import distance_buckets
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    d, H, G, D = z["width"], z["heads"], z["kv"], z["dim"]
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dtype=bf, k=1.0: (torch.randn(s, generator=g, device=dev) * k).to(dtype)     # noqa: E731
+    i32 = lambda a: torch.tensor(np.asarray(a), dtype=torch.int32, device=dev)                 # noqa: E731
+    hbm, tfl = peaks["hbm_gbs"], peaks["bf16_tflops"]
+    rows = {}
+
+    def note(name, ms, bytes_=0.0, flops=0.0):
+        r = {"us": round(ms * 1e3, 1)}
+        if bytes_:
+            r["gb_s"] = round(bytes_ / ms / 1e6, 1)
+            r["hbm_frac"] = round(bytes_ / ms / 1e6 / hbm, 3)
+        if flops:
+            r["tflops"] = round(flops / ms / 1e9, 1)
+            r["tensor_frac"] = round(flops / ms / 1e9 / tfl, 3)
+        rows[name] = r
+        print(f"[design_bench] {name}: {json.dumps(r)}", file=sys.stderr, flush=True)
+
+    def batch_ctx(q_lens, pos0, ps=16):
+        E_ = len(q_lens)
+        per = [-(-(p + n) // ps) for p, n in zip(pos0, q_lens)]
+        table = torch.full((E_, max(per)), -1, dtype=torch.int32)
+        at = 0
+        for e, n in enumerate(per):
+            table[e, :n] = torch.arange(at, at + n, dtype=torch.int32)
+            at += n
+        qs = np.concatenate([[0], np.cumsum(q_lens)[:-1]])
+        ctx = types.SimpleNamespace(
+            n_entries=E_, n_tokens=int(sum(q_lens)), max_q_len=max(q_lens), h_q_len=np.asarray(q_lens, dtype=np.int32),
+            h_pos0=np.asarray(pos0, dtype=np.int32), tok_entry=i32(np.repeat(np.arange(E_), q_lens)),
+            positions=i32(np.concatenate([p + np.arange(n) for p, n in zip(pos0, q_lens)])), entry_q_start=i32(qs),
+            entry_q_len=i32(q_lens), entry_pos0=i32(pos0), entry_slot=i32(np.arange(E_)), kv_bound=None)
+        return ctx, table.to(dev), at
+
+    rel = rnd(H, len(distance_buckets(32, z["bias_max"])), dtype=f32)
+    sinks, slopes = rnd(H, dtype=f32), torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], dtype=f32, device=dev)
+    rel2, sinks2 = rel * A.LOG2E, sinks * A.LOG2E
+    for label, q_lens, pos0 in (("prefill", [T], [0]), ("decode", [1] * batch, [context - 1] * batch)):
+        ctx, table, pages = batch_ctx(q_lens, pos0)
+        n, single = ctx.n_tokens, label == "decode"
+        # ---- attention with a soft cap, a distance table and sinks beside attention with a distance slope ----------
+        kc, vc = rnd(pages, G, 16, D), rnd(pages, G, 16, D)
+        kv = types.SimpleNamespace(k=kc, v=vc, page_size=16, group=0)
+        q, out = rnd(n, H * D), torch.empty(n, H * D, dtype=bf, device=dev)
+        pairs = T * (T + 1) / 2 if not single else batch * context
+        keys = T if not single else batch * context
+        bytes_, flops = 2.0 * G * 2 * D * keys + 4.0 * n * H * D, 2.0 * H * 2 * D * pairs
+        attend = lambda **kw: A.paged_attention_ex(ctx, q, out, kv, table, H, G, D, D, None, D ** -0.5, False, **kw)       # noqa: E731
+        note(f"capped_attention_{label}", timer(lambda: attend(rel=rel, rel_log2=rel2, sinks=sinks, sinks_log2=sinks2, softcap=30.0)), bytes_, flops)
+        note(f"table_bias_attention_{label}", timer(lambda: attend(rel=rel, rel_log2=rel2)), bytes_, flops)
+        note(f"slope_bias_attention_{label}", timer(lambda: attend(slopes=slopes)), bytes_, flops)
+        proj, qw, kw = rnd(n, (H + 2 * G) * D, dtype=f32), torch.ones(H * D, device=dev), torch.ones(G * D, device=dev)
+        prep = lambda **kw2: L.qk_prepare(proj, 0, H * D, (H + G) * D, 1, qw, kw, 1e-5, None, 1.0, ctx.positions, ctx.tok_entry, table, 16, q,   # noqa: E731
+                                          kc, vc, H, G, D, D, **kw2)
+        note(f"qk_prepare_temperature_{label}", timer(lambda: prep(temperature=(0.1, 1024), v_scale=0.9)), n * (H + 2 * G) * D * 6.0)
+        note(f"qk_prepare_{label}", timer(prep), n * (H + 2 * G) * D * 6.0)
+        # ---- the memories with decays per channel beside those with one per head -----------------------------------
+        rctx, _, _ = batch_ctx(q_lens, [0] * len(q_lens))
+        E, rank = len(q_lens), 64
+        args = (rctx.entry_q_start, rctx.entry_q_len, rctx.entry_slot, E)
+        Hd, Gd, Kd, Vd, taps = z["delta_heads"], z["delta_kv"], z["delta_dim"], z["delta_vdim"], z["taps"]
+        CH = 2 * Gd * Kd + Hd * Vd
+        cw, alog, nw = rnd(taps, CH, dtype=f32, k=0.4), rnd(Hd, dtype=f32, k=0.2), torch.ones(Vd, device=dev)
+        dtb, dtc = rnd(Hd, dtype=f32) - 3.0, rnd(Hd * Kd, dtype=f32) - 3.0
+        cp = rnd(n, CH + 2 * rank + Hd, dtype=f32, k=0.5)
+        a2, g2 = rnd(Hd * Kd, rank, k=0.1), rnd(Hd * Vd, rank, k=0.1)
+        state = torch.zeros(E, L.memory_state_floats("channel", Hd, Kd, Vd, taps, CH), device=dev)
+        so, dout = L.memory_tail_floats(taps, CH), torch.empty(n, Hd * Vd, dtype=bf, device=dev)
+        narrow = lambda: (L.low_rank(cp[:, CH:CH + rank], a2, "decay", dtc, alog), L.low_rank(cp[:, CH + rank:CH + 2 * rank], g2))       # noqa: E731
+        decay, gate = narrow()
+        cprep = lambda dec: L.channel_prepare(cp, 0, CH + 2 * rank, cw, dec, state, rctx.tok_entry, *args, Gd, Hd, Kd, Vd, single)       # noqa: E731
+        u, tab = cprep(decay)
+        cscan = lambda u_, t_: L.channel_scan(u_, t_, state, so, *args, Hd, Kd, Vd, single)       # noqa: E731
+        y = cscan(u, tab)
+
+        def whole_channel():
+            dec, gt = narrow()
+            L.memory_finish(cscan(*cprep(dec)), None, gt, "sigmoid", nw, 1e-5, dout, Hd, Vd)
+        least = n * (cp.shape[1] * 4.0 + Hd * Vd * 2.0) + 8.0 * state.numel()
+        work = 2.0 * n * Hd * Kd * Vd * 3
+        note(f"channel_delta_{label}", timer(whole_channel), least, work)
+        note(f"low_rank_two_{label}", timer(narrow), n * (2.0 * rank + Hd * Kd + Hd * Vd) * 4.0)
+        note(f"channel_prepare_{label}", timer(lambda: cprep(decay)), n * (CH + Hd * Kd + 3.25 * Hd * Kd + Hd * Vd) * 4.0)
+        note(f"channel_scan_{label}", timer(lambda: cscan(u, tab)), n * (3.25 * Hd * Kd + 2 * Hd * Vd) * 4.0 + 8.0 * E * Hd * Kd * Vd, work)
+        sp = rnd(n, CH + Hd * Vd + 2 * Hd, dtype=f32, k=0.5)
+        sprep = lambda: L.memory_prepare(sp, 0, CH + Hd * Vd + Hd, CH + Hd * Vd, cw, alog, dtb, state, rctx.tok_entry, *args, Gd, Hd, Kd, Vd, single)   # noqa: E731
+        su, st = sprep()
+        sscan = lambda u_, t_: L.delta_scan(u_, t_, state, so, *args, Hd, Gd, Kd, Vd, single)       # noqa: E731
+
+        def whole_delta():
+            L.memory_finish(sscan(*sprep()), None, sp[:, CH:CH + Hd * Vd], "silu", nw, 1e-5, dout, Hd, Vd)
+        note(f"delta_memory_{label}", timer(whole_delta), n * (sp.shape[1] * 4.0 + Hd * Vd * 2.0) + 8.0 * state.numel(), work)
+        note(f"memory_prepare_{label}", timer(sprep), n * CH * 8.0)
+        note(f"delta_scan_{label}", timer(lambda: sscan(su, st)), n * (CH + Hd * Vd) * 4.0 + 8.0 * E * Hd * Kd * Vd, work)
+        Hm, Km, Vm = z["mem_heads"], z["mem_dim"], z["mem_vdim"]
+        v0, gn = 2 * Hm * Km, torch.ones(Vm, device=dev)
+        dp, w2, b2 = rnd(n, v0 + 2 * Hm * Vm + rank, dtype=f32, k=0.5), rnd(Hm * Km, rank, k=0.1), rnd(Hm * Km, dtype=f32) + 2.0
+        mstate, mout = torch.zeros(E, L.memory_state_floats("gated", Hm, Km, Vm), device=dev), torch.empty(n, Hm * Vm, dtype=bf, device=dev)
+        dstate = torch.zeros(E, L.memory_state_floats("decayed", Hm, Km, Vm), device=dev)
+        alpha = L.low_rank(dp[:, v0 + 2 * Hm * Vm:], w2, "sigmoid", b2, tau=16.0)
+        dscan = lambda al: L.decayed_scan(dp, 0, Hm * Km, v0, al, dstate, 0, *args, Hm, Km, Vm, single)       # noqa: E731
+
+        def whole_decayed():
+            al = L.low_rank(dp[:, v0 + 2 * Hm * Vm:], w2, "sigmoid", b2, tau=16.0)
+            L.memory_finish(dscan(al), None, dp[:, v0 + Hm * Vm:v0 + 2 * Hm * Vm], "silu", gn, 1e-5, mout, Hm, Vm)
+        mwork = 2.0 * n * Hm * Km * Vm * 2
+        note(f"decayed_memory_{label}", timer(whole_decayed), n * (dp.shape[1] * 4.0 + Hm * Vm * 2.0) + 8.0 * dstate.numel(), mwork)
+        note(f"decayed_scan_{label}", timer(lambda: dscan(alpha)), n * (3 * Hm * Km + 2 * Hm * Vm) * 4.0 + 8.0 * dstate.numel(), mwork)
+        gp, gw = rnd(n, v0 + 2 * Hm * Vm + 2 * Hm, dtype=f32, k=0.5), torch.ones(Hm * Vm, device=dev)
+
+        def whole_gated():
+            y_, den = L.gated_scan(gp, 0, Hm * Km, v0, v0 + 2 * Hm * Vm, v0 + 2 * Hm * Vm + Hm, 15.0, mstate, 0, *args, Hm, Km, Vm, single)
+            L.memory_finish(y_, den, gp[:, v0 + Hm * Vm:v0 + 2 * Hm * Vm], "sigmoid", gw, 1e-5, mout, Hm, Vm)
+        note(f"gated_memory_{label}", timer(whole_gated), n * (gp.shape[1] * 4.0 + Hm * Vm * 2.0) + 8.0 * mstate.numel(), mwork)
+        # ---- latent attention over a window with sinks beside latent attention over all keys -----------------------
+        Hl, Dl, Rl, Vl, C, W = z["lat_heads"], z["lat_dim"], z["lat_rot"], z["lat_vdim"], z["lat_rank"], z["window"]
+        lkv = types.SimpleNamespace(k=rnd(pages, 1, 16, C + Rl), v=None, page_size=16, group=0)
+        rows_h = -(-n // 128) * 128
+        q_lat, q_rot, o_lat = rnd(Hl, rows_h, C, dtype=f32), rnd(Hl, rows_h, Rl, dtype=f32), torch.empty(Hl, rows_h, C, dtype=bf, device=dev)
+        lsink = rnd(Hl, dtype=f32)
+        lsink2 = lsink * A.LOG2E
+        seen = sum(min(i + 1, W) for i in range(T)) if not single else batch * min(context, W)
+        for name, p, kk, kw2 in (("window_sink_latent", seen, T if not single else batch * min(context, W), dict(window=W, sinks=lsink, sinks_log2=lsink2)),
+                                 ("latent", pairs, keys, {})):
+            ms = timer(lambda: LA.attention(ctx, q_lat, q_rot, o_lat, lkv, table, n, Hl, C, Rl, (Dl + Rl) ** -0.5, **kw2))
+            note(f"{name}_attention_{label}", ms, 2.0 * (C + Rl) * kk + n * Hl * (4.0 * (C + Rl) + 2.0 * C), 2.0 * Hl * (2 * C + Rl) * p)
+        # ---- a norm on a sublayer's result beside norms on both sides; the embedding; the feed-forward ---------------
+        x, yv, w1 = rnd(n, d, dtype=f32), rnd(n, d, dtype=f32), torch.ones(d, device=dev)
+        hb = torch.empty(n, d, dtype=bf, device=dev)
+        one = K.NormedDelta(yv, w1, 1e-5)
+        note(f"post_norm_{label}", timer(lambda: L.sandwich_norm(x, one, None, 0.0, hb)), n * d * (4 + 4 + 4 + 2.0))
+        note(f"sandwich_norm_{label}", timer(lambda: L.sandwich_norm(x, one, w1, 1e-5, hb)), n * d * (4 + 4 + 4 + 2.0))
+        tabl, ids = rnd(z["vocab"], d), i32(np.arange(n) % z["vocab"])
+        compose = lambda **kw2: L.embed_compose(tabl, ids, x, 1.0, None, None, None, None, rctx.positions, rctx.tok_entry, *args, single, **kw2)   # noqa: E731
+        note(f"embed_norm_{label}", timer(lambda: compose(norm_w=w1, eps=1e-5, h=hb)), n * d * (2 + 4 + 2.0))
+        note(f"embed_gather_{label}", timer(lambda: K.embed_gather(tabl, ids, x)), n * d * 6.0)
+        ff = z["ff"]
+        act, wgu, wdn, bgu = torch.empty(n, ff, dtype=bf, device=dev), rnd(2 * ff, d, k=0.02), rnd(d, ff, k=0.02), rnd(2 * ff, dtype=f32)
+        for name, bias in (("biased_swiglu", bgu), ("swiglu", None)):
+            lin, dn = Linear(wgu, bias), Linear(wdn, None)
+
+            def mlp():
+                if not lin.forward_swiglu(hb, act):
+                    if bias is not None:
+                        L.glu_act(lin.forward(hb, defer=True), act)
+                    else:
+                        K.swiglu(lin.forward(hb, defer=True), act)
+                dn.forward(act, defer=True, residual=True)
+            note(f"{name}_{label}", timer(mlp), 3.0 * d * ff * 2, 2.0 * n * 3 * d * ff)
+    return rows
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="design_bench")
-    ap.add_argument("--design", default="vufizen", choices=["vufizen", "gositar", "banelix", "pibavik", "nuvarax"])
+    ap.add_argument("--design", default="vufizen", choices=["vufizen", "gositar", "banelix", "pibavik", "nuvarax", "dukolorn"])
     ap.add_argument("--sizes", default="s,m")
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--context", type=int, default=2048)
@@ -938,7 +1126,8 @@ def main(argv=None) -> int:
         "pibavik": (PIBAVIK_SIZES, pibavik_config, {"banelix": banelix_beside_pibavik}, time_pibavik_kernels),
         "nuvarax": (NUVARAX_SIZES, nuvarax_config, {"pibavik": lambda z, n: pibavik_config(PIBAVIK_SIZES[z["beside"]], n),
                                                     "banelix": lambda z, n: banelix_beside_pibavik(PIBAVIK_SIZES[z["beside"]], n)},
-                    time_nuvarax_kernels)}[args.design]
+                    time_nuvarax_kernels),
+        "dukolorn": (DUKOLORN_SIZES, dukolorn_config, {"nuvarax": nuvarax_config}, time_dukolorn_kernels)}[args.design]
     out = {"bench": "designs", "design": args.design, "dtype": "bf16", "data": "synthetic", "prompt": args.prompt, "context": args.context,
            "batch": args.batch, "layers": args.layers, "peaks": peaks, "sizes": {}}
     for name in [s for s in args.sizes.split(",") if s]:

@@ -107,3 +107,20 @@ def test_design_bench_of_nuvarax(capsys):
             "gated_memory_prefill", "gated_memory_decode", "sandwich_norm_prefill", "sandwich_norm_with_conv_decode",
             "input_conv_prefill", "embed_compose_decode"} <= set(rows)
     assert all(r["us"] > 0 for r in rows.values())
+
+
+def test_design_bench_of_dukolorn(capsys):
+    """``bench.py --designs --design dukolorn`` at a size made for tests: beside Nuvarax, the closest design."""
+    import json
+    from infero_b200.tools import design_bench
+    assert design_bench.main(["--design", "dukolorn", "--sizes", "t", "--prompt", "600", "--context", "300", "--batch", "3",
+                              "--layers", "4", "--kernels-at", "t"]) == 0
+    line = json.loads(capsys.readouterr().out.strip().splitlines()[-1])
+    assert line["design"] == "dukolorn" and set(line["sizes"]["t"]) == {"shape", "dukolorn", "nuvarax"}
+    for design in ("dukolorn", "nuvarax"):
+        assert line["sizes"]["t"][design]["prefill_tok_s"] > 0 and line["sizes"]["t"][design]["decode_tok_s"] > 0
+    rows = line["kernels"]["rows"]
+    assert {"capped_attention_prefill", "capped_attention_decode", "channel_delta_prefill", "channel_delta_decode", "decayed_memory_prefill",
+            "decayed_memory_decode", "window_sink_latent_attention_prefill", "post_norm_decode", "embed_norm_prefill",
+            "biased_swiglu_decode"} <= set(rows)
+    assert all(r["us"] > 0 for r in rows.values())
