@@ -426,6 +426,22 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     TL_END(TL_GEMM);
 }
 
+// (A row of sixteen biases: vector loads where they are 32-bit and aligned; every lane reads the same ones.)
+__device__ __forceinline__ void add_bias16(float* v, const void* __restrict__ bias, int bias_dtype, int at, int end) {
+    const float* b = (const float*)bias + at;
+    if (bias_dtype == INFERO_F32 && at + 16 <= end && (reinterpret_cast<uintptr_t>(b) & 15u) == 0) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float4 f = __ldg(reinterpret_cast<const float4*>(b) + e);
+            v[4 * e] += f.x, v[4 * e + 1] += f.y, v[4 * e + 2] += f.z, v[4 * e + 3] += f.w;
+        }
+        return;
+    }
+#pragma unroll
+    for (int e = 0; e < 16; ++e)
+        if (at + e < end) v[e] += load_any(bias, bias_dtype, at + e);
+}
+
 // One epilogue warp's share of a finished accumulator: its 32 rows (TMEM lanes at lane_addr, result
 // row ra for this thread) by BN columns starting at feature b0, written as the epilogue EPI says.
 template <int EPI, typename OutT>
@@ -451,11 +467,7 @@ __device__ __forceinline__ void drain_accumulator(uint32_t lane_addr, int ra, in
                 if (EPI == EPI_ROW_SWIGLU) {
                     OutT* dst = out + (size_t)ra * ldc + (rb >> 1);
                     float h[8];
-                    if (bias) {
-#pragma unroll
-                        for (int e = 0; e < 16; ++e)
-                            if (rb + e < RB) v[e] += load_any(bias, bias_dtype, rb + e);
-                    }
+                    if (bias) add_bias16(v, bias, bias_dtype, rb, RB);
 #pragma unroll
                     for (int e = 0; e < 8; ++e)
                         h[e] = act_kind == GLU_SILU ? silu_mul(v[2 * e], v[2 * e + 1])
@@ -475,11 +487,7 @@ __device__ __forceinline__ void drain_accumulator(uint32_t lane_addr, int ra, in
                     }
                 } else {
                     OutT* dst = out + (size_t)ra * ldc + rb;
-                    if (bias) {
-#pragma unroll
-                        for (int e = 0; e < 16; ++e)
-                            if (rb + e < RB) v[e] += load_any(bias, bias_dtype, rb + e);
-                    }
+                    if (bias) add_bias16(v, bias, bias_dtype, rb, RB);
                     if (act_kind == ACT_RELU2) {
 #pragma unroll
                         for (int e = 0; e < 16; ++e) {

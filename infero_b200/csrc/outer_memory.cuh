@@ -426,31 +426,31 @@ __global__ void __launch_bounds__(288) memory_scan_kernel(const ScanArgs a) {
                     }
                 }
                 scatter_sum<ND, LG>(dots, lane);
+                // the lanes are shared out among the columns; each collects the sums of its own and solves for its u's
                 using At = Scattered<ND, LG>;
-                float all[ND];
+                constexpr int PER = At::per_lane, STR = At::stride, SHARE = LG / CPT;
+                const int mine = CPT > 1 ? l / SHARE : 0;
+                float all[2 * C];
 #pragma unroll
-                for (int i = 0; i < ND; ++i)
-                    all[i] = LG == 1 ? dots[i] : __shfl_sync(0xffffffffu, dots[i % At::per_lane], i / At::per_lane * At::stride, LG);
-                float u[CPT][C], G = 1.f;            // u_i times the decays of the tokens behind it; the product of all decays
+                for (int i = 0; i < 2 * C; ++i)
+                    all[i] = LG == 1 ? dots[i] : __shfl_sync(0xffffffffu, dots[i % PER], mine * (2 * C / PER * STR) + i / PER * STR, LG);
+                float u[C], G = 1.f;                 // u_i times the decays of the tokens behind it; the product of all decays
 #pragma unroll
                 for (int j = 0; j < C; ++j) {
                     const float4 g = gb[(t0 + j) * 3], p0 = gb[(t0 + j) * 3 + 1], p1 = gb[(t0 + j) * 3 + 2];
                     const float kk[3] = {p0.y, p0.w, p1.y}, kq[3] = {p0.z, p1.x, p1.z};
                     if constexpr (RULE == RULE_DELTA) G *= g.x;
+                    float b = G * all[j], o = G * all[C + j];
 #pragma unroll
-                    for (int p = 0; p < CPT; ++p) {
-                        float b = G * all[p * 2 * C + j], o = G * all[p * 2 * C + C + j];
-#pragma unroll
-                        for (int i = 0; i < j; ++i) {
-                            // (channel: the decays in between are in the products and in what is written)
-                            if constexpr (RULE == RULE_DELTA) u[p][i] *= g.x;
-                            b = fmaf(kk[(j - i - 1) % 3], u[p][i], b);
-                            o = fmaf(kq[(j - i - 1) % 3], u[p][i], o);
-                        }
-                        u[p][j] = g.y * (vb[(t0 + j) * COLS + p] - b);
-                        o = fmaf(p0.x, u[p][j], o);
-                        if (l == 0) yb[(t0 + j) * COLS + p] = o;
+                    for (int i = 0; i < j; ++i) {
+                        // (channel: the decays in between are in the products and in what is written)
+                        if constexpr (RULE == RULE_DELTA) u[i] *= g.x;
+                        b = fmaf(kk[(j - i - 1) % 3], u[i], b);
+                        o = fmaf(kq[(j - i - 1) % 3], u[i], o);
                     }
+                    u[j] = g.y * (vb[(t0 + j) * COLS + mine] - b);
+                    o = fmaf(p0.x, u[j], o);
+                    if (l % SHARE == 0) yb[(t0 + j) * COLS + mine] = o;
                 }
                 if constexpr (RULE == RULE_DELTA) {
                     const f2 decay = f2_of(G, G);
@@ -473,7 +473,10 @@ __global__ void __launch_bounds__(288) memory_scan_kernel(const ScanArgs a) {
                 for (int j = 0; j < C; ++j) {
                     f2 uu[CPT];
 #pragma unroll
-                    for (int p = 0; p < CPT; ++p) uu[p] = f2_of(u[p][j], u[p][j]);
+                    for (int p = 0; p < CPT; ++p) {
+                        const float up = CPT > 1 ? __shfl_sync(0xffffffffu, u[j], p * SHARE, LG) : u[j];
+                        uu[p] = f2_of(up, up);
+                    }
 #pragma unroll
                     for (int n = 0; n < NR / 4; ++n) {
                         ulonglong2 fw;
@@ -557,49 +560,34 @@ __global__ void __launch_bounds__(288) memory_scan_kernel(const ScanArgs a) {
 
 inline bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
-// INFERO_MEMORY_COLUMNS (1 or 2) forces how many columns a thread of the rules with decays per channel holds in portions.
-inline int forced_columns() {
-    static const int v = [] { const char* e = getenv("INFERO_MEMORY_COLUMNS"); return e ? atoi(e) : 0; }();
-    return v;
-}
-
 template <int RULE>
 int launch_scan(ScanArgs a, int n_entries, bool single, int sm_count, cudaStream_t stream) {
-    constexpr bool WIDER = ScanPlan<RULE>::aux;      // rules whose portions have instances with two columns a thread
     // Few columns: eight numbers a thread, so that there are warps enough to hide one another's latencies; many: sixteen, so
     // that fewer threads read the same keys and queries.  Portions run best in small blocks, single tokens (one round trip to
     // memory for the whole state) in large ones.
-    int NR = a.K > 256 || (long long)n_entries * a.H * a.W * a.K > 300000 ? 16 : 8;
-    if (WIDER && a.K <= 64) NR = 8;                  // (no instances of sixteen for few lanes)
+    const int NR = a.K > 256 || (long long)n_entries * a.H * a.W * a.K > 300000 ? 16 : 8;
     int LG = 1;
     while (LG * NR < a.K) LG *= 2;
     const int sms = sm_count > 0 ? sm_count : 148;
     int threads = single ? (NR == 16 ? 128 : 256) : 64;
     while (threads < 4 * LG) threads *= 2;
     while (threads > 32 && threads / 2 >= 4 * LG && (long long)n_entries * a.H * ((a.W + threads / LG - 1) / (threads / LG)) < sms) threads /= 2;
-    const int CPT = WIDER && !single ? (forced_columns() ? forced_columns() : 1) : 1;
-    const int COLS = threads / LG * CPT;
+    const int COLS = threads / LG;
     const dim3 grid(n_entries, a.H, (a.W + COLS - 1) / COLS);
     INFERO_REQUIRE(grid.z <= 65535, "memory_scan: %d columns are too many for one launch", a.W);
     a.wide = a.wide && a.V % 4 == 0 && a.v_off % 4 == 0 && COLS % 4 == 0;
     const size_t smem = ScanPlan<RULE>::smem_floats(NR * LG, COLS) * sizeof(float);
 #define GO(R, L)                                                                                                       \
     do {                                                                                                               \
-        auto k = single ? memory_scan_kernel<RULE, R, L, 1, 1>                                                         \
-                        : CPT > 1 ? memory_scan_kernel<RULE, R, L, GROUP, WIDER ? 2 : 1> : memory_scan_kernel<RULE, R, L, GROUP, 1>; \
+        auto k = single ? memory_scan_kernel<RULE, R, L, 1, 1> : memory_scan_kernel<RULE, R, L, GROUP, 1>;             \
         if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
         /* a portion's blocks run long: started under the kernel in front, they would crowd on the first free SMs */        \
         if (single) launch_pdl(k, grid, dim3(threads + 32), smem, stream, a);                                          \
         else k<<<grid, threads + 32, smem, stream>>>(a);                                                               \
     } while (0)
 #define PICK(L)                                                                                                        \
-    if constexpr (!WIDER || L >= 8) {                                                                                  \
-        if (NR == 16) {                                                                                                \
-            GO(16, L);                                                                                                 \
-            break;                                                                                                     \
-        }                                                                                                              \
-    }                                                                                                                  \
-    GO(8, L);                                                                                                          \
+    if (NR == 16) GO(16, L);                                                                                           \
+    else GO(8, L);                                                                                                     \
     break
     switch (LG) {
         case 1: PICK(1);
@@ -610,6 +598,48 @@ int launch_scan(ScanArgs a, int n_entries, bool single, int sm_count, cudaStream
         default: PICK(32);
     }
 #undef PICK
+#undef GO
+    return infero_check_launch("memory_scan");
+}
+
+// The rules with decays per channel read three vectors a token, so a thread takes few rows of several columns: what it reads
+// serves them all, and a reduction over more lanes costs little more when it carries several columns' sums.  Enough warps to keep
+// the schedulers busy come first (INFERO_MEMORY_COLUMNS = 1, 2 or 4 forces the columns of a portion).
+inline int forced_columns() {
+    static const int v = [] { const char* e = getenv("INFERO_MEMORY_COLUMNS"); return e ? atoi(e) : 0; }();
+    return v;
+}
+
+template <int RULE>
+int launch_channel_scan(ScanArgs a, int n_entries, bool single, int sm_count, cudaStream_t stream) {
+    const int NR = a.K <= 128 ? 4 : a.K <= 256 ? 8 : 16, LG = a.K <= 32 ? 8 : a.K <= 64 ? 16 : 32;
+    const int sms = sm_count > 0 ? sm_count : 148;
+    auto blocks = [&](int cols) { return (long long)n_entries * a.H * ((a.W + cols - 1) / cols); };
+    int CPT = 4;
+    while (CPT > 1 && blocks(32 / LG * CPT) < 2 * sms) CPT /= 2;         // (blocks of one warp: warps)
+    if (single) CPT = CPT == 4 ? 4 : 1;
+    else if (forced_columns() == 1 || forced_columns() == 2 || forced_columns() == 4) CPT = forced_columns();
+    int threads = single ? 256 : 128;
+    while (threads > 32 && threads / 2 / LG * CPT >= 4 && blocks(threads / LG * CPT) * 5 < 4 * sms) threads /= 2;
+    const int COLS = threads / LG * CPT;
+    const dim3 grid(n_entries, a.H, (a.W + COLS - 1) / COLS);
+    INFERO_REQUIRE(grid.z <= 65535, "memory_scan: %d columns are too many for one launch", a.W);
+    a.wide = a.wide && a.V % 4 == 0 && a.v_off % 4 == 0 && COLS % 4 == 0;
+    const size_t smem = ScanPlan<RULE>::smem_floats(NR * LG, COLS) * sizeof(float);
+#define GO(R, L)                                                                                                       \
+    do {                                                                                                               \
+        auto k = single ? (CPT == 4 ? memory_scan_kernel<RULE, R, L, 1, 4> : memory_scan_kernel<RULE, R, L, 1, 1>)      \
+                        : CPT == 4 ? memory_scan_kernel<RULE, R, L, GROUP, 4>                                          \
+                        : CPT == 2 ? memory_scan_kernel<RULE, R, L, GROUP, 2> : memory_scan_kernel<RULE, R, L, GROUP, 1>; \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+        if (single) launch_pdl(k, grid, dim3(threads + 32), smem, stream, a);                                          \
+        else k<<<grid, threads + 32, smem, stream>>>(a);                                                               \
+    } while (0)
+    if (NR == 4 && LG == 8) GO(4, 8);
+    else if (NR == 4 && LG == 16) GO(4, 16);
+    else if (NR == 4) GO(4, 32);
+    else if (NR == 8) GO(8, 32);
+    else GO(16, 32);
 #undef GO
     return infero_check_launch("memory_scan");
 }

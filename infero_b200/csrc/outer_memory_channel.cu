@@ -40,7 +40,8 @@ __device__ __forceinline__ void conv_group(const PrepareArgs& a, int t, int nt, 
         if (j < nt) conv_silu<VEC>(a, t + j, first, tail, c, v[j]);
 }
 
-// A warp per (token, head); it works where the token starts a group of its request's new tokens.
+// A warp per (token, unit) where the token starts a group of its request's new tokens; a unit is the q and k of a kv head, worked
+// out for every head that reads them, or the v of a head.  In steps of single tokens it also moves its channels' tails on.
 template <int VEC, int NV>
 __global__ void __launch_bounds__(PREP_WARPS * 32) channel_prepare_kernel(const ChannelArgs ca) {
     const PrepareArgs& a = ca.p;
@@ -48,23 +49,39 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) channel_prepare_kernel(const 
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * PREP_WARPS + warp;
-    if (item >= (long long)a.n_tokens * a.H) return;
-    const int t = (int)(item / a.H), h = (int)(item % a.H);
+    const int units = a.G + a.H;
+    if (item >= (long long)a.n_tokens * units) return;
+    const int t = (int)(item / units), unit = (int)(item % units);
     const int e = a.tok_entry[t], first = a.entry_q_start[e];
     if ((t - first) % GROUP) return;
     const int nt = min(GROUP, first + ca.entry_q_len[e] - t);
     float* tail = a.state + (long long)a.entry_slot[e] * a.state_stride;
-    const int HK = a.H * a.K, kvh = h / (a.H / a.G), cq = kvh * a.K, ck = (a.G + kvh) * a.K, cv = 2 * a.G * a.K + h * a.V;
+    const int HK = a.H * a.K;
     const long long U = 4ll * HK + (long long)a.H * a.V;
-    float* ur = a.u + t * U + (size_t)h * a.K;           // this head's columns of the group's first row
+    if (unit >= a.G) {
+        const int h = unit - a.G;
+        float* vr = a.u + t * U + 4ll * HK + (size_t)h * a.V;
+        for (int i = lane * VEC; i < a.V; i += 32 * VEC) {
+            float v[GROUP][VEC];
+            conv_group<VEC>(a, t, nt, first, tail, 2 * a.G * a.K + h * a.V + i, v);
+#pragma unroll
+            for (int j = 0; j < GROUP; ++j)
+                if (j < nt) put<VEC>(vr + j * U + i, v[j]);
+        }
+        if (lane < nt) {
+            const float b = sigmoid_f(a.proj[(size_t)(t + lane) * a.proj_stride + a.step_off + h]);
+            *reinterpret_cast<float4*>(a.table + ((size_t)h * a.n_tokens + t + lane) * DELTA_ROW) = make_float4(1.f, b, 0.f, 0.f);
+        }
+        return;
+    }
     float q[NV][GROUP][VEC], k[NV][GROUP][VEC];
     float sums[2 * GROUP] = {};
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
         const int i = (n * 32 + lane) * VEC;
         if (i < a.K) {
-            conv_group<VEC>(a, t, nt, first, tail, cq + i, q[n]);
-            conv_group<VEC>(a, t, nt, first, tail, ck + i, k[n]);
+            conv_group<VEC>(a, t, nt, first, tail, unit * a.K + i, q[n]);
+            conv_group<VEC>(a, t, nt, first, tail, (a.G + unit) * a.K + i, k[n]);
 #pragma unroll
             for (int j = 0; j < GROUP; ++j)
 #pragma unroll
@@ -76,114 +93,108 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) channel_prepare_kernel(const 
     }
     scatter_sum<2 * GROUP, 32>(sums, lane);
     const float q_scale = 1.0f / sqrtf((float)a.K);
-    float rq[GROUP], rk[GROUP];
 #pragma unroll
     for (int j = 0; j < GROUP; ++j) {
-        rq[j] = 1.0f / sqrtf(__shfl_sync(0xffffffffu, sums[0], 4 * j) + 1e-6f) * q_scale;
-        rk[j] = 1.0f / sqrtf(__shfl_sync(0xffffffffu, sums[0], 4 * (GROUP + j)) + 1e-6f);
-    }
-    // 0 .. 3: k_j . q_j; then, over the pairs (0,1) (1,2) (2,3) (0,2) (1,3) (0,3), k_i . k_j and k_i . q_j with the decays between
-    float dots[16] = {};
+        const float rq = 1.0f / sqrtf(__shfl_sync(0xffffffffu, sums[0], 4 * j) + 1e-6f) * q_scale;
+        const float rk = 1.0f / sqrtf(__shfl_sync(0xffffffffu, sums[0], 4 * (GROUP + j)) + 1e-6f);
 #pragma unroll
-    for (int n = 0; n < NV; ++n) {
-        const int i = (n * 32 + lane) * VEC;
-        if (i < a.K) {
-            float g[GROUP][VEC];
+        for (int n = 0; n < NV; ++n)
+            if ((n * 32 + lane) * VEC < a.K) {
 #pragma unroll
-            for (int j = 0; j < GROUP; ++j) {
-#pragma unroll
-                for (int r = 0; r < VEC; ++r) g[j][r] = 1.f;
-                if (j < nt) {
-                    const float* src = ca.g + (size_t)(t + j) * HK + (size_t)h * a.K + i;
-                    if constexpr (VEC == 4) load4f(src, g[j]);
-                    else g[j][0] = src[0];
-                }
-#pragma unroll
-                for (int r = 0; r < VEC; ++r) q[n][j][r] *= rq[j], k[n][j][r] *= rk[j];
+                for (int r = 0; r < VEC; ++r) q[n][j][r] *= rq, k[n][j][r] *= rk;
             }
-            float all[VEC], w[GROUP][VEC];               // the decays up to here; D_j k_j
+    }
+    const int per = a.H / a.G;
+    for (int h = unit * per; h < (unit + 1) * per; ++h) {
+        float* ur = a.u + t * U + (size_t)h * a.K;       // this head's columns of the group's first row
+        // 0 .. 3: k_j . q_j; then, over the pairs (0,1) (1,2) (2,3) (0,2) (1,3) (0,3), k_i . k_j and k_i . q_j with the decays
+        // between
+        float dots[16] = {};
 #pragma unroll
-            for (int r = 0; r < VEC; ++r) all[r] = 1.f;
+        for (int n = 0; n < NV; ++n) {
+            const int i = (n * 32 + lane) * VEC;
+            if (i < a.K) {
+                float g[GROUP][VEC];
 #pragma unroll
-            for (int j = 0; j < GROUP; ++j) {
-                float gq[VEC], gk[VEC];
+                for (int j = 0; j < GROUP; ++j) {
 #pragma unroll
-                for (int r = 0; r < VEC; ++r) {
-                    all[r] *= g[j][r];
-                    gq[r] = all[r] * q[n][j][r];
-                    gk[r] = all[r] * k[n][j][r];
-                    dots[j] = fmaf(k[n][j][r], q[n][j][r], dots[j]);
-                    w[j][r] = k[n][j][r];
-                }
-#pragma unroll
-                for (int b = 0; b < j; ++b) {            // the tokens before it in the group: pair (b, j), j - b tokens back
-                    constexpr int at[GROUP] = {0, 0, 3, 5};
-                    const int c = at[j - b] + b;
-#pragma unroll
-                    for (int r = 0; r < VEC; ++r) {
-                        w[b][r] *= g[j][r];
-                        dots[4 + c] = fmaf(w[b][r], k[n][j][r], dots[4 + c]);
-                        dots[10 + c] = fmaf(w[b][r], q[n][j][r], dots[10 + c]);
+                    for (int r = 0; r < VEC; ++r) g[j][r] = 1.f;
+                    if (j < nt) {
+                        const float* src = ca.g + (size_t)(t + j) * HK + (size_t)h * a.K + i;
+                        if constexpr (VEC == 4) load4f(src, g[j]);
+                        else g[j][0] = src[0];
                     }
                 }
-                if (j < nt) {
-                    put<VEC>(ur + j * U + i, gq);
-                    put<VEC>(ur + j * U + HK + i, gk);
+                float all[VEC], w[GROUP][VEC];           // the decays up to here; D_j k_j
+#pragma unroll
+                for (int r = 0; r < VEC; ++r) all[r] = 1.f;
+#pragma unroll
+                for (int j = 0; j < GROUP; ++j) {
+                    float gq[VEC], gk[VEC];
+#pragma unroll
+                    for (int r = 0; r < VEC; ++r) {
+                        all[r] *= g[j][r];
+                        gq[r] = all[r] * q[n][j][r];
+                        gk[r] = all[r] * k[n][j][r];
+                        dots[j] = fmaf(k[n][j][r], q[n][j][r], dots[j]);
+                        w[j][r] = k[n][j][r];
+                    }
+#pragma unroll
+                    for (int b = 0; b < j; ++b) {        // the tokens before it in the group: pair (b, j), j - b tokens back
+                        constexpr int at[GROUP] = {0, 0, 3, 5};
+                        const int c = at[j - b] + b;
+#pragma unroll
+                        for (int r = 0; r < VEC; ++r) {
+                            w[b][r] *= g[j][r];
+                            dots[4 + c] = fmaf(w[b][r], k[n][j][r], dots[4 + c]);
+                            dots[10 + c] = fmaf(w[b][r], q[n][j][r], dots[10 + c]);
+                        }
+                    }
+                    if (j < nt) {
+                        put<VEC>(ur + j * U + i, gq);
+                        put<VEC>(ur + j * U + HK + i, gk);
+                    }
                 }
+#pragma unroll
+                for (int j = 0; j < GROUP; ++j)
+                    if (j < nt) put<VEC>(ur + j * U + 2 * HK + i, w[j]);
+                put<VEC>(ur + (nt - 1) * U + 3 * HK + i, all);
             }
-#pragma unroll
-            for (int j = 0; j < GROUP; ++j)
-                if (j < nt) put<VEC>(ur + j * U + 2 * HK + i, w[j]);
-            put<VEC>(ur + (nt - 1) * U + 3 * HK + i, all);
         }
-    }
-    scatter_sum<16, 32>(dots, lane);                     // value m in lane 2 m
-    float* table = a.table + ((size_t)h * a.n_tokens + t) * DELTA_ROW;
-    if (!(lane & 1)) {
-        const int m = lane >> 1, c = m < 10 ? m - 4 : m - 10, back = c < 3 ? 1 : c < 5 ? 2 : 3;
-        const int j = m < 4 ? m : (back == 1 ? c : back == 2 ? c - 3 : 0) + back;
-        if (j < nt) table[j * DELTA_ROW + (m < 4 ? 4 : (m < 10 ? 3 : 4) + 2 * back)] = dots[0];
-    } else if (lane < 2 * nt) {
-        const int j = lane >> 1;
-        const float b = sigmoid_f(a.proj[(size_t)(t + j) * a.proj_stride + a.step_off + h]);
-        *reinterpret_cast<float4*>(table + j * DELTA_ROW) = make_float4(1.f, b, 0.f, 0.f);
-    }
-    float* vr = a.u + t * U + 4ll * HK + (size_t)h * a.V;
-    for (int i = lane * VEC; i < a.V; i += 32 * VEC) {
-        float v[GROUP][VEC];
-        conv_group<VEC>(a, t, nt, first, tail, cv + i, v);
-#pragma unroll
-        for (int j = 0; j < GROUP; ++j)
-            if (j < nt) put<VEC>(vr + j * U + i, v[j]);
+        scatter_sum<16, 32>(dots, lane);                 // value m in lane 2 m
+        if (!(lane & 1)) {
+            const int m = lane >> 1, c = m < 10 ? m - 4 : m - 10, back = c < 3 ? 1 : c < 5 ? 2 : 3;
+            const int j = m < 4 ? m : (back == 1 ? c : back == 2 ? c - 3 : 0) + back;
+            if (j < nt) a.table[((size_t)h * a.n_tokens + t + j) * DELTA_ROW + (m < 4 ? 4 : (m < 10 ? 3 : 4) + 2 * back)] = dots[0];
+        }
     }
 }
 
 }  // namespace
 
 int memory::scan_channel(const ScanArgs& a, int n_entries, bool single, int sm_count, cudaStream_t stream) {
-    return launch_scan<RULE_CHANNEL>(a, n_entries, single, sm_count, stream);
+    return launch_channel_scan<RULE_CHANNEL>(a, n_entries, single, sm_count, stream);
 }
 
 extern "C" {
 
-// The channel rule's prepare: u [T, 4 H K + H V], table [H, T, 12], g [T, H K] the decays (see ChannelArgs).  move_tail: every
-// request of the step brings one token and H == G, so that the tails are moved on here; else by infero_conv_tail.
+// The channel rule's prepare: u [T, 4 H K + H V], table [H, T, 12], g [T, H K] the decays (see ChannelArgs).  single: every
+// request of the step brings one token; the tails are moved on here then, else by infero_conv_tail.
 int infero_channel_prepare(const float* proj, long long proj_stride, int x_off, const float* conv_w, int taps, float* state,
                            long long state_stride, const int* tok_entry, const int* entry_q_start, const int* entry_q_len,
                            const int* entry_slot, float* u, float* table, const float* g, int step_off, int n_tokens, int G, int H,
-                           int K, int V, int move_tail, cudaStream_t stream) {
+                           int K, int V, int single, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     INFERO_REQUIRE(taps >= 1 && taps <= MAX_TAPS, "channel_prepare: %d taps outside 1..%d", taps, MAX_TAPS);
     INFERO_REQUIRE(K >= 1 && K <= MAX_K && V >= 1 && G >= 1 && H % G == 0, "channel_prepare: %d heads over %d of %d x %d", H, G, K, V);
-    INFERO_REQUIRE(!move_tail || H == G, "channel_prepare: several heads share a tail");
     ChannelArgs c = {};
     PrepareArgs& a = c.p;
     a.proj = proj, a.proj_stride = proj_stride, a.conv_w = conv_w, a.state = state, a.state_stride = state_stride;
     a.tok_entry = tok_entry, a.entry_q_start = entry_q_start, a.entry_slot = entry_slot, a.u = u, a.table = table;
     a.step_off = step_off, a.x_off = x_off, a.taps = taps, a.n_tokens = n_tokens, a.G = G, a.H = H, a.K = K, a.V = V;
-    a.CH = 2 * G * K + H * V, a.move_tail = move_tail;
+    a.CH = 2 * G * K + H * V, a.move_tail = single;
     c.g = g, c.entry_q_len = entry_q_len;
-    const long long items = (long long)n_tokens * H;
+    const long long items = (long long)n_tokens * (G + H);
     const dim3 grid((unsigned)((items + PREP_WARPS - 1) / PREP_WARPS)), block(PREP_WARPS * 32);
     const bool vec = K % 4 == 0 && V % 4 == 0 && proj_stride % 4 == 0 && x_off % 4 == 0 && state_stride % 4 == 0 && al16(proj) &&
                      al16(conv_w) && al16(state) && al16(u) && al16(g);

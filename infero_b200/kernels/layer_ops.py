@@ -698,19 +698,26 @@ LOW_RANK_MODES = {"plain": 0, "decay": 1, "sigmoid": 2}
 
 
 def low_rank(a: torch.Tensor, w: torch.Tensor, mode: str = "plain", bias: Optional[torch.Tensor] = None,
-             a_log: Optional[torch.Tensor] = None, tau: float = 1.0) -> torch.Tensor:
+             a_log: Optional[torch.Tensor] = None, tau: float = 1.0, beside=None):
     """float32 [T, N] from a product's narrow middle ``a`` (float32 [T, R], a column slice) and w [N, R]: z = a w^T (+ bias);
-    "decay": exp(-exp(a_log of the head) softplus(z)) with N / len(a_log) columns a head; "sigmoid": sigmoid(z)^(1 / tau)."""
+    "decay": exp(-exp(a_log of the head) softplus(z)) with N / len(a_log) columns a head; "sigmoid": sigmoid(z)^(1 / tau).
+    ``beside`` = (a2, w2): a second, plain product from columns of the same rows, in the same launch; both are returned then."""
     T, R = a.shape
     N = w.shape[0]
     assert a.dtype == torch.float32 and a.stride(1) == 1 and w.is_contiguous() and w.shape[1] == R
     assert bias is None or bias.numel() == N
     assert mode != "decay" or N % a_log.numel() == 0
     out = torch.empty((T, N), dtype=torch.float32, device=a.device)
+    a2 = w2 = out2 = None
+    if beside is not None:
+        a2, w2 = beside
+        assert a2.dtype == torch.float32 and a2.stride() == a.stride() and a2.shape[0] == T and w2.is_contiguous() and w2.shape[1] == a2.shape[1]
+        out2 = torch.empty((T, w2.shape[0]), dtype=torch.float32, device=a.device)
     _check(lib().infero_low_rank(_ptr(a), c_longlong(a.stride(0)), _ptr(w), c_int(_dt(w)), _ptr(_f32(bias, "bias")), _ptr(_f32(a_log, "a_log")),
                                  c_int(N // a_log.numel() if a_log is not None else 1), c_float(tau), c_int(LOW_RANK_MODES[mode]), _ptr(out),
-                                 c_int(T), c_int(N), c_int(R), _stream()))
-    return out
+                                 c_int(T), c_int(N), c_int(R), _ptr(a2), _ptr(w2), c_int(_dt(w2) if w2 is not None else 0), _ptr(out2),
+                                 c_int(w2.shape[0] if w2 is not None else 0), c_int(w2.shape[1] if w2 is not None else 0), _stream()))
+    return out if out2 is None else (out, out2)
 
 
 def channel_prepare(proj: torch.Tensor, x_off: int, step_off: int, conv_w: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
@@ -727,11 +734,10 @@ def channel_prepare(proj: torch.Tensor, x_off: int, step_off: int, conv_w: torch
     table = torch.empty((H, T, 12), dtype=torch.float32, device=proj.device)
     L = lib()
     batch = (_ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")))
-    own_tail = single and H == G
     _check(L.infero_channel_prepare(_ptr(proj), c_longlong(proj.stride(0)), c_int(x_off), _ptr(_f32(conv_w, "conv_w")), c_int(taps), _ptr(state),
                                     c_longlong(state.stride(0)), _ptr(_i32(tok_entry, "tok_entry")), *batch, _ptr(u), _ptr(table), _ptr(decay),
-                                    c_int(step_off), c_int(T), c_int(G), c_int(H), c_int(K), c_int(V), c_int(1 if own_tail else 0), _stream()))
-    if not own_tail:
+                                    c_int(step_off), c_int(T), c_int(G), c_int(H), c_int(K), c_int(V), c_int(1 if single else 0), _stream()))
+    if not single:
         _check(L.infero_conv_tail(_ptr(proj[:, x_off:]), c_int(proj.stride(0)), c_int(taps), _ptr(state), c_longlong(state.stride(0)), *batch,
                                   c_int(n_entries), c_int(CH), _stream()))
     return u, table

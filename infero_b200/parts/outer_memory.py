@@ -257,8 +257,8 @@ class ChannelDeltaMemory(_ChannelDecayed):
     def core(self, ctx, proj: torch.Tensor, off: int, slot, out: torch.Tensor, scale: float = 1.0) -> None:
         H, G, K, V = self.H, self.G, self.K, self.V
         state, single = ctx.state(slot.cache), single_tokens(ctx)
-        decay = L.low_rank(self._narrow(proj, off, "decay_down"), self.decay_up, "decay", self.dt_bias, self.a_log)
-        gate = L.low_rank(self._narrow(proj, off, "gate_down"), self.gate_up)
+        decay, gate = L.low_rank(self._narrow(proj, off, "decay_down"), self.decay_up, "decay", self.dt_bias, self.a_log,
+                                 beside=(self._narrow(proj, off, "gate_down"), self.gate_up))
         batch = (ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries)
         u, table = L.channel_prepare(proj, off, off + self.off["step"], self.conv_w, decay, state, ctx.tok_entry, *batch, G, H, K, V, single)
         y = L.channel_scan(u, table, state, self.s_off, *batch, H, K, V, single)

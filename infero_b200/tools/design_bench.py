@@ -1013,7 +1013,7 @@ def time_dukolorn_kernels(z, T, context, batch, timer, peaks):
         a2, g2 = rnd(Hd * Kd, rank, k=0.1), rnd(Hd * Vd, rank, k=0.1)
         state = torch.zeros(E, L.memory_state_floats("channel", Hd, Kd, Vd, taps, CH), device=dev)
         so, dout = L.memory_tail_floats(taps, CH), torch.empty(n, Hd * Vd, dtype=bf, device=dev)
-        narrow = lambda: (L.low_rank(cp[:, CH:CH + rank], a2, "decay", dtc, alog), L.low_rank(cp[:, CH + rank:CH + 2 * rank], g2))       # noqa: E731
+        narrow = lambda: L.low_rank(cp[:, CH:CH + rank], a2, "decay", dtc, alog, beside=(cp[:, CH + rank:CH + 2 * rank], g2))       # noqa: E731
         decay, gate = narrow()
         cprep = lambda dec: L.channel_prepare(cp, 0, CH + 2 * rank, cw, dec, state, rctx.tok_entry, *args, Gd, Hd, Kd, Vd, single)       # noqa: E731
         u, tab = cprep(decay)

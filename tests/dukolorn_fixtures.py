@@ -18,7 +18,7 @@ _TMP = tempfile.mkdtemp(prefix="infero_b200_dukolorn_")
 # at most one in twenty above the second.  (A norm over a memory's read-out turns a read-out that happens to be near zero into
 # a direction, which 16 bits do not hold: rounding nothing but the sublayers' inputs and results to bf16 in the plain
 # statement moves single rows of these models by up to 0.22, half of the rows by less than 0.01.)
-TOL = {"float32": (1e-4, 2e-5), "bfloat16": (0.4, 0.06)}
+TOL = {"float32": (5e-4, 2e-5), "bfloat16": (0.4, 0.06)}
 
 
 def delta(heads, kv, dim, vdim, conv):

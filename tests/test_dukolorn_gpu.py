@@ -78,6 +78,9 @@ def test_decays_and_gates_through_a_narrow_middle(T, H, K, rank, wd):
         want = torch.sigmoid(z + b.double()) ** (1.0 / tau)
         got = L.low_rank(da, dw, "sigmoid", b.to(DEV), tau=tau).cpu().double()
         assert float((got - want).abs().max()) < 5e-6 and bool((got <= 1).all())
+    w2 = torch.randn(2 * H * K + 3, 5, generator=g).to(wd)                          # two products of the same rows in one launch
+    one, two = L.low_rank(da, dw, beside=(rows.to(DEV)[:, :5], w2.to(DEV)))
+    assert _rel(one, z) < 2e-6 and _rel(two, rows[:, :5].double() @ w2.double().T) < 2e-6
 
 
 # ---- the two memories ----------------------------------------------------------------------------------------------------
@@ -179,9 +182,9 @@ def test_a_state_lasts_for_hundreds_of_tokens(rule):
         assert _rel(plain(h2)[-1:], want[-1:]) > 0.005
 
 
-@pytest.mark.parametrize("columns", ["1", "2"])
-def test_portions_with_one_and_with_two_columns_a_thread(columns):
-    """The scans have both forms; each in a process of its own, since the choice is read once."""
+@pytest.mark.parametrize("columns", ["1", "2", "4"])
+def test_portions_with_one_two_and_four_columns_a_thread(columns):
+    """The scans have all three forms; each in a process of its own, since the choice is read once."""
     import os
     import subprocess
     import sys
