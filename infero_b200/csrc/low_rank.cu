@@ -3,7 +3,8 @@
 //   z[t, n] = sum_r a[t, r] w[n, r] (+ bias[n])          a: columns of an input product's 32-bit rows
 //   PLAIN    out = z
 //   DECAY    out = exp(-exp(a_log[n / per_head]) softplus(z))
-//   SIGMOID  out = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
+//   SIGMOID  out = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau), alone or as the first part of the records [decays | k | q] of a
+//            recurrence's scan (channel_memory.cuh), q and k copied from columns of the same rows
 //
 // The middle is a few dozen wide, so the result is bound by its own size; a block makes a tile of tokens by 64 columns,
 // both operands transposed in shared memory.  Sums run over r in ascending order, one fused multiply-add each, whatever the
@@ -26,6 +27,11 @@ struct LowRankArgs {
     long long a_stride;
     int w_bf16, T, N, R, mode, per_head;
     float inv_tau;
+    // records: rec [N / per_head, T, 3 row_len], row_len >= per_head (the rows behind are zero); k and q at these columns of qk
+    float* rec;
+    const float* qk;
+    long long qk_stride;
+    int q_off, k_off, row_len;
 };
 
 // four neighbouring numbers of a row of w, zeros beyond its end
@@ -113,6 +119,30 @@ __global__ void __launch_bounds__(THREADS) low_rank_kernel(const LowRankArgs fir
             const float z = acc[i][j] + bias[j];
             v[j] = p.mode == LR_PLAIN ? z : expf(rate[j] * softplus_f(p.mode == LR_DECAY ? z : -z));
         }
+        if (p.rec) {
+            const float* row = p.qk + t * p.qk_stride;
+            if constexpr (PN == 4) {
+                const int n = n0 + tn, h = n / p.per_head, c = n - h * p.per_head;
+                if (n + 3 < p.N && ((p.per_head | p.q_off | p.k_off | (int)p.qk_stride) & 3) == 0 && c + 4 < p.per_head) {
+                    float* r = p.rec + ((size_t)h * p.T + t) * 3 * p.row_len + c;
+                    *reinterpret_cast<float4*>(r) = make_float4(v[0], v[1], v[2], v[3]);
+                    *reinterpret_cast<float4*>(r + p.row_len) = *reinterpret_cast<const float4*>(row + p.k_off + n);
+                    *reinterpret_cast<float4*>(r + 2 * p.row_len) = *reinterpret_cast<const float4*>(row + p.q_off + n);
+                    continue;
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < PN; ++j) {
+                const int n = n0 + tn + j;
+                if (n >= p.N) break;
+                const int h = n / p.per_head, c = n - h * p.per_head;
+                float* r = p.rec + ((size_t)h * p.T + t) * 3 * p.row_len;
+                r[c] = v[j], r[p.row_len + c] = row[p.k_off + n], r[2 * p.row_len + c] = row[p.q_off + n];
+                if (c == p.per_head - 1)
+                    for (int i = p.per_head; i < p.row_len; ++i) r[i] = r[p.row_len + i] = r[2 * p.row_len + i] = 0.f;
+            }
+            continue;
+        }
         if constexpr (PN == 4) {
             if (vec && n0 + tn + 3 < p.N) {
                 *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
@@ -155,6 +185,23 @@ int infero_low_rank(const float* a, long long a_stride, const void* w, int w_dty
     if (TM == 64) launch_pdl(low_rank_kernel<64>, grid, dim3(THREADS), 0, stream, p, q);
     else launch_pdl(low_rank_kernel<8>, grid, dim3(THREADS), 0, stream, p, q);
     return infero_check_launch("low_rank");
+}
+
+// Decays sigmoid(z)^(1 / tau) as records [N / K, T, 3 row_len] with k and q from columns of qk's rows (16-byte aligned).
+int infero_low_rank_records(const float* a, long long a_stride, const void* w, int w_dtype, const float* bias, float tau, float* rec,
+                            int row_len, const float* qk, long long qk_stride, int q_off, int k_off, int T, int H, int K, int R,
+                            cudaStream_t stream) {
+    if (T == 0) return 0;
+    LowRankArgs p = {};
+    if (make_args(p, a, a_stride, w, w_dtype, bias, nullptr, K, tau, LR_SIGMOID, rec, T, H * K, R)) return 1;
+    INFERO_REQUIRE(row_len >= K && row_len % 4 == 0 && (reinterpret_cast<uintptr_t>(qk) & 15u) == 0, "low_rank: rows of %d for %d", row_len, K);
+    p.rec = rec, p.qk = qk, p.qk_stride = qk_stride, p.q_off = q_off, p.k_off = k_off, p.row_len = row_len;
+    const int TM = T > 32 ? 64 : 8;
+    const dim3 grid((H * K + TN - 1) / TN, (T + TM - 1) / TM);
+    INFERO_REQUIRE(grid.y <= 65535, "low_rank: %d tokens in one launch", T);
+    if (TM == 64) launch_pdl(low_rank_kernel<64>, grid, dim3(THREADS), 0, stream, p, p);
+    else launch_pdl(low_rank_kernel<8>, grid, dim3(THREADS), 0, stream, p, p);
+    return infero_check_launch("low_rank_records");
 }
 
 }  // extern "C"

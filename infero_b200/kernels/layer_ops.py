@@ -592,7 +592,7 @@ def embed_compose(table: torch.Tensor, ids: torch.Tensor, out_x: torch.Tensor, s
 
 
 # ---- recurrences with a matrix per head (csrc/outer_memory.cu) -------------------------------------------------------
-MEMORY_RULES = {"delta": 0, "gated": 1, "channel": 2, "decayed": 3}
+MEMORY_RULES = {"delta": 0, "gated": 1}
 
 
 def memory_tail_floats(taps: int, channels: int) -> int:
@@ -652,7 +652,7 @@ def memory_gates(gates: torch.Tensor, in_off: int, forget_off: int, cap: float, 
 
 
 def _memory_scan(rule: str, src, q_off, k_off, v_off, table, gates, in_off, forget_off, cap, q_scale, state, s_off, entry_q_start,
-                 entry_q_len, entry_slot, n_entries, H, G, K, V, single, aux=None, group_decay=None):
+                 entry_q_len, entry_slot, n_entries, H, G, K, V, single):
     from .tc_gemm import sm_count
     T = src.shape[0]
     gated = rule == "gated"
@@ -667,7 +667,7 @@ def _memory_scan(rule: str, src, q_off, k_off, v_off, table, gates, in_off, forg
         c_float(q_scale), _ptr(state), c_longlong(state.stride(0)), c_longlong(s_off),
         _ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")),
         _ptr(y), _ptr(den), c_int(n_entries), c_int(1 if single else 0), c_int(H), c_int(G), c_int(K), c_int(V),
-        c_int(sm_count(src.device)), _ptr(aux), _ptr(group_decay), c_longlong(aux.stride(0) if aux is not None else 0), _stream()))
+        c_int(sm_count(src.device)), _stream()))
     return y, den
 
 
@@ -693,7 +693,7 @@ def gated_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, in_off: i
                         entry_q_start, entry_q_len, entry_slot, n_entries, H, H, K, V, single)
 
 
-# ---- memories with a decay per channel of a key (csrc/low_rank.cu, outer_memory_channel.cu, outer_memory_decayed.cu) -------
+# ---- memories with a decay per channel of a key (csrc/low_rank.cu, channel_memory.cuh) -------------------------------
 LOW_RANK_MODES = {"plain": 0, "decay": 1, "sigmoid": 2}
 
 
@@ -720,45 +720,72 @@ def low_rank(a: torch.Tensor, w: torch.Tensor, mode: str = "plain", bias: Option
     return out if out2 is None else (out, out2)
 
 
+def decayed_records(a: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, tau: float, proj: torch.Tensor, q_off: int, k_off: int, H: int,
+                    K: int) -> torch.Tensor:
+    """What the scan of gated linear attention reads: records [H, T, 3 Kp] of a token's decays sigmoid(a w^T + bias)^(1 / tau), its k
+    and its q (columns of the 32-bit product rows ``proj``)."""
+    T, R = a.shape
+    assert a.dtype == proj.dtype == torch.float32 and a.stride(1) == proj.stride(1) == 1 and w.is_contiguous() and tuple(w.shape) == (H * K, R)
+    assert bias.numel() == H * K and proj.shape[1] >= max(q_off, k_off) + H * K
+    Kp = int(lib().infero_channel_rows(c_int(K)))
+    rec = torch.empty((H, T, 3 * Kp), dtype=torch.float32, device=a.device)
+    _check(lib().infero_low_rank_records(_ptr(a), c_longlong(a.stride(0)), _ptr(w), c_int(_dt(w)), _ptr(_f32(bias, "bias")), c_float(tau), _ptr(rec),
+                                         c_int(Kp), _ptr(proj), c_longlong(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(T), c_int(H),
+                                         c_int(K), c_int(R), _stream()))
+    return rec
+
+
 def channel_prepare(proj: torch.Tensor, x_off: int, step_off: int, conv_w: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
                     tok_entry, entry_q_start, entry_q_len, entry_slot, n_entries: int, G: int, H: int, K: int, V: int, single: bool):
-    """What the delta rule's scan needs where every channel of a key decays on its own: (u [T, 4 H K + H V], table [H, T, 12])
-    from the 32-bit product rows ([q | k | v] at ``x_off``, raw steps at ``step_off``) and the decays [T, H K]; see
-    csrc/outer_memory_channel.cu.  The requests' tails (the convolution's last taps - 1 inputs) move on."""
+    """What the delta rule's scan needs where every channel of a key decays on its own: (values [T, H V], records [H, slots, n] of
+    groups of four tokens) from the 32-bit product rows ([q | k | v] at ``x_off``, raw steps at ``step_off``) and the decays
+    [T, H K]; see csrc/channel_memory.cuh.  The requests' tails (the convolution's last taps - 1 inputs) move on."""
     T = proj.shape[0]
     taps, CH = conv_w.shape
     assert CH == 2 * G * K + H * V and proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= max(x_off + CH, step_off + H)
     assert decay.dtype == torch.float32 and decay.is_contiguous() and tuple(decay.shape) == (T, H * K)
     assert state.dtype == torch.float32 and state.is_contiguous()
-    u = torch.empty((T, 4 * H * K + H * V), dtype=torch.float32, device=proj.device)
-    table = torch.empty((H, T, 12), dtype=torch.float32, device=proj.device)
     L = lib()
+    slots = int(L.infero_delta_slots(c_int(T), c_int(n_entries)))
+    v = torch.empty((T, H * V), dtype=torch.float32, device=proj.device)
+    rec = torch.empty((H, slots, int(L.infero_delta_record(c_int(K)))), dtype=torch.float32, device=proj.device)
     batch = (_ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")))
     _check(L.infero_channel_prepare(_ptr(proj), c_longlong(proj.stride(0)), c_int(x_off), _ptr(_f32(conv_w, "conv_w")), c_int(taps), _ptr(state),
-                                    c_longlong(state.stride(0)), _ptr(_i32(tok_entry, "tok_entry")), *batch, _ptr(u), _ptr(table), _ptr(decay),
-                                    c_int(step_off), c_int(T), c_int(G), c_int(H), c_int(K), c_int(V), c_int(1 if single else 0), _stream()))
+                                    c_longlong(state.stride(0)), _ptr(_i32(tok_entry, "tok_entry")), *batch, _ptr(v), _ptr(rec), c_int(slots),
+                                    _ptr(decay), c_int(step_off), c_int(T), c_int(G), c_int(H), c_int(K), c_int(V), c_int(1 if single else 0),
+                                    _stream()))
     if not single:
         _check(L.infero_conv_tail(_ptr(proj[:, x_off:]), c_int(proj.stride(0)), c_int(taps), _ptr(state), c_longlong(state.stride(0)), *batch,
                                   c_int(n_entries), c_int(CH), _stream()))
-    return u, table
+    return v, rec
 
 
-def channel_scan(u: torch.Tensor, table: torch.Tensor, state: torch.Tensor, s_off: int, entry_q_start, entry_q_len, entry_slot,
+def _channel_scan(f, rec, n, v, extra, state, s_off, entry_q_start, entry_q_len, entry_slot, n_entries, H, K, V, single):
+    from .tc_gemm import sm_count
+    assert rec.is_contiguous() and rec.dtype == v.dtype == torch.float32 and v.stride(1) == 1 and v.shape[1] == H * V
+    assert state.dtype == torch.float32 and state.is_contiguous() and s_off + H * V * K <= state.shape[1]
+    y = torch.empty((v.shape[0], H * V), dtype=torch.float32, device=v.device)
+    _check(f(_ptr(rec), c_int(n), _ptr(v), c_longlong(v.stride(0)), *extra, _ptr(state), c_longlong(state.stride(0)), c_longlong(s_off),
+             _ptr(_i32(entry_q_start, "entry_q_start")), _ptr(_i32(entry_q_len, "entry_q_len")), _ptr(_i32(entry_slot, "entry_slot")), _ptr(y),
+             c_int(n_entries), c_int(1 if single else 0), c_int(H), c_int(K), c_int(V), c_int(sm_count(v.device)), _stream()))
+    return y
+
+
+def channel_scan(v: torch.Tensor, rec: torch.Tensor, state: torch.Tensor, s_off: int, entry_q_start, entry_q_len, entry_slot,
                  n_entries: int, H: int, K: int, V: int, single: bool = False) -> torch.Tensor:
     """The delta rule with a decay per channel, from what ``channel_prepare`` left; float32 [T, H V].  S [H, V, K] at ``s_off``."""
-    HK = H * K
-    assert table.is_contiguous() and tuple(table.shape) == (H, u.shape[0], 12) and u.shape[1] == 4 * HK + H * V
-    return _memory_scan("channel", u, 0, HK, 4 * HK, table, None, 0, 0, 0.0, 1.0, state, s_off, entry_q_start, entry_q_len, entry_slot,
-                        n_entries, H, H, K, V, single, aux=u[:, 2 * HK:], group_decay=u[:, 3 * HK:])[0]
+    assert rec.shape[0] == H
+    return _channel_scan(lib().infero_channel_scan, rec, rec.shape[1], v, (), state, s_off, entry_q_start, entry_q_len, entry_slot, n_entries,
+                         H, K, V, single)
 
 
-def decayed_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, state: torch.Tensor, s_off: int, entry_q_start,
-                 entry_q_len, entry_slot, n_entries: int, H: int, K: int, V: int, single: bool = False) -> torch.Tensor:
-    """Gated linear attention of every request over its new tokens, from the 32-bit product rows and the decays [T, H K];
-    float32 [T, H V], q times K^-1/2.  S [H, V, K] at ``s_off``."""
-    assert decay.dtype == torch.float32 and decay.is_contiguous() and tuple(decay.shape) == (proj.shape[0], H * K)
-    return _memory_scan("decayed", proj, q_off, k_off, v_off, None, None, 0, 0, 0.0, K ** -0.5, state, s_off, entry_q_start, entry_q_len,
-                        entry_slot, n_entries, H, H, K, V, single, aux=decay)[0]
+def decayed_scan(v: torch.Tensor, rec: torch.Tensor, state: torch.Tensor, s_off: int, entry_q_start, entry_q_len, entry_slot,
+                 n_entries: int, H: int, K: int, V: int, single: bool = False) -> torch.Tensor:
+    """Gated linear attention of every request over its new tokens, from the values (columns of the product's rows) and
+    ``decayed_records``; float32 [T, H V], q times K^-1/2.  S [H, V, K] at ``s_off``."""
+    assert tuple(rec.shape[:2]) == (H, v.shape[0])
+    return _channel_scan(lib().infero_decayed_scan, rec, rec.shape[1], v, (c_float(K ** -0.5),), state, s_off, entry_q_start, entry_q_len,
+                         entry_slot, n_entries, H, K, V, single)
 
 
 def memory_finish(y: torch.Tensor, den: Optional[torch.Tensor], gate: torch.Tensor, act: str, norm_w: torch.Tensor, eps: float,

@@ -184,7 +184,7 @@ def reduce_partials(partial: torch.Tensor, bias: Optional[torch.Tensor], out: to
 def error_flag() -> int:
     """Synchronises; non-zero if a kernel gave up on one of its bounded waits since the flag was last
     read (reading clears it).  1-3: a product kernel, 4: decode attention, 5-7: prompt attention,
-    8: the many-row norm."""
+    8: the many-row norm, 9: the scan of a memory with decays per channel."""
     return int(lib().infero_tc_error_flag())
 
 

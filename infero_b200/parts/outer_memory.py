@@ -235,7 +235,7 @@ class ChannelDeltaMemory(_ChannelDecayed):
                 ("gate_down", self.ranks["gate_down"]), ("step", self.H)]
 
     def state_spec(self) -> Optional[StateSpec]:
-        return StateSpec((L.memory_state_floats("channel", self.H, self.K, self.V, self.taps, self.CH),), torch.float32)
+        return StateSpec((L.memory_state_floats("delta", self.H, self.K, self.V, self.taps, self.CH),), torch.float32)
 
     def declare(self) -> List[TensorDecl]:
         d, r = self.spec.hidden, self.ranks
@@ -260,14 +260,14 @@ class ChannelDeltaMemory(_ChannelDecayed):
         decay, gate = L.low_rank(self._narrow(proj, off, "decay_down"), self.decay_up, "decay", self.dt_bias, self.a_log,
                                  beside=(self._narrow(proj, off, "gate_down"), self.gate_up))
         batch = (ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries)
-        u, table = L.channel_prepare(proj, off, off + self.off["step"], self.conv_w, decay, state, ctx.tok_entry, *batch, G, H, K, V, single)
-        y = L.channel_scan(u, table, state, self.s_off, *batch, H, K, V, single)
+        v, rec = L.channel_prepare(proj, off, off + self.off["step"], self.conv_w, decay, state, ctx.tok_entry, *batch, G, H, K, V, single)
+        y = L.channel_scan(v, rec, state, self.s_off, *batch, H, K, V, single)
         L.memory_finish(y, None, gate, "sigmoid", self.norm_w, float(self.spec.norm_eps), out, H, V, scale)
 
 
 class DecayedMemory(_ChannelDecayed):
     """Gated linear attention: S <- diag(a) S + k v^T, o = S^T q, with decays a = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau) per key
-    channel and every head its own q and k.  One input product gives [q | k | v | gate | decay's middle]; ``low_rank`` (decays)
+    channel and every head its own q and k.  One input product gives [q | k | v | gate | decay's middle]; ``decayed_records`` (decays beside k and q)
     -> ``decayed_scan`` -> ``memory_finish`` (RMS norm with a weight shared by the heads, silu gate) -> output product.  The
     request's state: S."""
 
@@ -284,7 +284,7 @@ class DecayedMemory(_ChannelDecayed):
                 ("decay_down", self.ranks["decay_down"])]
 
     def state_spec(self) -> Optional[StateSpec]:
-        return StateSpec((L.memory_state_floats("decayed", self.H, self.K, self.V),), torch.float32)
+        return StateSpec((L.memory_state_floats("delta", self.H, self.K, self.V),), torch.float32)
 
     def declare(self) -> List[TensorDecl]:
         return self._declare_rows() + [
@@ -301,8 +301,9 @@ class DecayedMemory(_ChannelDecayed):
 
     def core(self, ctx, proj: torch.Tensor, off: int, slot, out: torch.Tensor, scale: float = 1.0) -> None:
         H, K, V, o = self.H, self.K, self.V, self.off
-        decay = L.low_rank(self._narrow(proj, off, "decay_down"), self.decay_up, "sigmoid", self.decay_bias, tau=float(self.spec.decay_tau))
-        y = L.decayed_scan(proj, off + o["q"], off + o["k"], off + o["v"], decay, ctx.state(slot.cache), 0, ctx.entry_q_start, ctx.entry_q_len,
+        rec = L.decayed_records(self._narrow(proj, off, "decay_down"), self.decay_up, self.decay_bias, float(self.spec.decay_tau), proj,
+                                off + o["q"], off + o["k"], H, K)
+        y = L.decayed_scan(proj[:, off + o["v"]:off + o["v"] + H * V], rec, ctx.state(slot.cache), 0, ctx.entry_q_start, ctx.entry_q_len,
                            ctx.entry_slot, ctx.n_entries, H, K, V, single_tokens(ctx))
         L.memory_finish(y, None, proj[:, off + o["gate"]:off + o["gate"] + H * V], "silu", self.norm_w, float(self.spec.norm_eps), out,
                         H, V, scale)

@@ -1011,7 +1011,7 @@ def time_dukolorn_kernels(z, T, context, batch, timer, peaks):
         dtb, dtc = rnd(Hd, dtype=f32) - 3.0, rnd(Hd * Kd, dtype=f32) - 3.0
         cp = rnd(n, CH + 2 * rank + Hd, dtype=f32, k=0.5)
         a2, g2 = rnd(Hd * Kd, rank, k=0.1), rnd(Hd * Vd, rank, k=0.1)
-        state = torch.zeros(E, L.memory_state_floats("channel", Hd, Kd, Vd, taps, CH), device=dev)
+        state = torch.zeros(E, L.memory_state_floats("delta", Hd, Kd, Vd, taps, CH), device=dev)
         so, dout = L.memory_tail_floats(taps, CH), torch.empty(n, Hd * Vd, dtype=bf, device=dev)
         narrow = lambda: L.low_rank(cp[:, CH:CH + rank], a2, "decay", dtc, alog, beside=(cp[:, CH + rank:CH + 2 * rank], g2))       # noqa: E731
         decay, gate = narrow()
@@ -1043,16 +1043,17 @@ def time_dukolorn_kernels(z, T, context, batch, timer, peaks):
         v0, gn = 2 * Hm * Km, torch.ones(Vm, device=dev)
         dp, w2, b2 = rnd(n, v0 + 2 * Hm * Vm + rank, dtype=f32, k=0.5), rnd(Hm * Km, rank, k=0.1), rnd(Hm * Km, dtype=f32) + 2.0
         mstate, mout = torch.zeros(E, L.memory_state_floats("gated", Hm, Km, Vm), device=dev), torch.empty(n, Hm * Vm, dtype=bf, device=dev)
-        dstate = torch.zeros(E, L.memory_state_floats("decayed", Hm, Km, Vm), device=dev)
-        alpha = L.low_rank(dp[:, v0 + 2 * Hm * Vm:], w2, "sigmoid", b2, tau=16.0)
-        dscan = lambda al: L.decayed_scan(dp, 0, Hm * Km, v0, al, dstate, 0, *args, Hm, Km, Vm, single)       # noqa: E731
+        dstate = torch.zeros(E, L.memory_state_floats("delta", Hm, Km, Vm), device=dev)
+        records = lambda: L.decayed_records(dp[:, v0 + 2 * Hm * Vm:], w2, b2, 16.0, dp, 0, Hm * Km, Hm, Km)       # noqa: E731
+        dscan = lambda r: L.decayed_scan(dp[:, v0:v0 + Hm * Vm], r, dstate, 0, *args, Hm, Km, Vm, single)       # noqa: E731
+        rec = records()
 
         def whole_decayed():
-            al = L.low_rank(dp[:, v0 + 2 * Hm * Vm:], w2, "sigmoid", b2, tau=16.0)
-            L.memory_finish(dscan(al), None, dp[:, v0 + Hm * Vm:v0 + 2 * Hm * Vm], "silu", gn, 1e-5, mout, Hm, Vm)
+            L.memory_finish(dscan(records()), None, dp[:, v0 + Hm * Vm:v0 + 2 * Hm * Vm], "silu", gn, 1e-5, mout, Hm, Vm)
         mwork = 2.0 * n * Hm * Km * Vm * 2
         note(f"decayed_memory_{label}", timer(whole_decayed), n * (dp.shape[1] * 4.0 + Hm * Vm * 2.0) + 8.0 * dstate.numel(), mwork)
-        note(f"decayed_scan_{label}", timer(lambda: dscan(alpha)), n * (3 * Hm * Km + 2 * Hm * Vm) * 4.0 + 8.0 * dstate.numel(), mwork)
+        note(f"decayed_records_{label}", timer(records), n * (5 * Hm * Km + rank) * 4.0)
+        note(f"decayed_scan_{label}", timer(lambda: dscan(rec)), n * (3 * Hm * Km + 2 * Hm * Vm) * 4.0 + 8.0 * dstate.numel(), mwork)
         gp, gw = rnd(n, v0 + 2 * Hm * Vm + 2 * Hm, dtype=f32, k=0.5), torch.ones(Hm * Vm, device=dev)
 
         def whole_gated():
