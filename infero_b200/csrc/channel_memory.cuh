@@ -8,8 +8,8 @@
 // is one contiguous piece of memory and one bulk copy:
 //
 //   delta rule, a record per group of four tokens of a request: [G | table | token 0 | .. | token 3], G [Kp] the product of the
-//     group's decays, table 4 x 12 floats (1, beta, two unused; k . q; and, 1, 2 and 3 tokens back in the group, k_back . k and
-//     k_back . q with the decays in between; one unused), a token [G_j k_j | G_j q_j | D_j k_j] with G_j the product of the decays up
+//     group's decays, table 4 x 8 floats (beta; k . q; and, 1, 2 and 3 tokens back in the group, k_back . k and k_back . q with the
+//     decays in between), a token [G_j k_j | G_j q_j | D_j k_j] with G_j the product of the decays up
 //     to it and D_j that of the tokens behind it.  All factors are at most one; nothing is divided.  A group that is not full is
 //     filled up with tokens of zeros.  Request e's groups start at slot (its first row) / 4 + e.
 //   gated linear attention, a record per token: [decays | k | q].
@@ -17,7 +17,8 @@
 // Kp is K rounded up to what the lanes hold, the rows behind K zero.  A block owns (request, head, a block of columns); a thread
 // holds NR rows of CPT neighbouring columns in registers for the whole portion, so that what it reads of a token serves all of
 // them.  Four tokens are taken together: the sums over the lanes of all of them are formed at once, and the delta rule's u's
-// follow by forward substitution from the products in the table, the lanes shared out among the columns.  A helper warp brings
+// follow by forward substitution from the products in the table, the lanes shared out among the columns (a lane keeps its columns
+// in an order of its own, the one that it ends up with first, so that the exchanges need no selection).  A helper warp brings
 // the stages in, two ahead.  Groups are counted from a request's own first new token: a token's arithmetic does not depend on the
 // batch, nor beyond rounding on how its prompt was cut.  Steps of single tokens run the same code in groups of one.
 #pragma once
@@ -26,7 +27,7 @@
 
 namespace memory {
 
-constexpr int TABLE = GROUP * DELTA_ROW;             // floats of a group's table
+constexpr int TOKEN_ROW = 8, TABLE = GROUP * TOKEN_ROW;       // floats of a token in a group's table
 
 inline int padded_rows(int K) { return K <= 32 ? 32 : K <= 64 ? 64 : K <= 128 ? 128 : K <= 256 ? 256 : 512; }
 __host__ __device__ inline int delta_record(int Kp) { return (1 + 3 * GROUP) * Kp + TABLE; }
@@ -45,6 +46,7 @@ struct ChannelScanArgs {
     float q_scale;
 };
 
+template <int N> __device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void bulk_copy(void* dst_smem, const void* src, uint32_t bytes, uint64_t* bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(tc::smem_u32(dst_smem)),
                  "l"(src), "r"(bytes), "r"(tc::smem_u32(bar)) : "memory");
@@ -52,22 +54,27 @@ __device__ __forceinline__ void bulk_copy(void* dst_smem, const void* src, uint3
 
 template <bool DELTA, int Kp, int C> struct ChannelPlan {
     static constexpr int TPS = C == 1 ? 1 : Kp > 256 ? 4 : 8;                            // tokens a stage holds
+    static constexpr int RING = C == 1 ? 1 : 3;                                     // stages: one at hand, the others on their way
     static constexpr int REC = DELTA ? (1 + 3 * C) * Kp + TABLE : 3 * Kp;                // floats read of a record
     static constexpr int STAGE = DELTA ? TPS / C * REC : TPS * REC;
-    static size_t smem_bytes(int cols) { return ((size_t)STAGES * (STAGE + TPS * cols)) * sizeof(float); }
+    // (behind the stages: every warp's u's, written twice, in two turns)
+    static size_t smem_bytes(int cols) { return ((size_t)RING * (STAGE + TPS * cols) + (DELTA ? 4 * C * cols : 0)) * sizeof(float); }
 };
+
+template <int N> struct Int { static constexpr int value = N; };
 
 template <bool DELTA, int NR, int LG, int C, int CPT>
 __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs a) {
-    constexpr int Kp = NR * LG, NP = NR / 2, N4 = NR / 4, SHARE = LG / CPT;
+    constexpr int Kp = NR * LG, NP = NR / 2, N4 = NR / 4, SHARE = LG / CPT, V4 = 3 * Kp / 4;
     using Plan = ChannelPlan<DELTA, Kp, C>;
     constexpr int TPS = Plan::TPS, REC = Plan::REC;
     extern __shared__ __align__(128) float sm[];
-    __shared__ __align__(8) uint64_t full[STAGES];
+    __shared__ __align__(8) uint64_t full[Plan::RING];
     __shared__ int never;
     const int nc = blockDim.x - 32;                  // threads that hold columns
     const int COLS = nc / LG * CPT;
-    float* vs = sm + STAGES * Plan::STAGE;           // [STAGES][TPS][COLS]
+    float* vs = sm + Plan::RING * Plan::STAGE;           // [Plan::RING][TPS][COLS]
+    f2* us = reinterpret_cast<f2*>(vs + Plan::RING * TPS * COLS);         // [2][COLS][C] the u's, twice each
     pdl_launch_dependents();
     const int e = blockIdx.x, h = blockIdx.y, pb = blockIdx.z;
     const int n_new = a.entry_q_len[e];
@@ -77,7 +84,7 @@ __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs
     float* S_head = a.state + (long long)a.entry_slot[e] * a.state_stride + a.s_off + (size_t)h * a.V * a.K;
     if (tid == 0) {
         never = 0;
-        for (int i = 0; i < STAGES; ++i) tc::mbar_init(&full[i], 1);
+        for (int i = 0; i < Plan::RING; ++i) tc::mbar_init(&full[i], 1);
         tc::fence_barrier_init();
         tc::fence_proxy_async();
     }
@@ -90,7 +97,7 @@ __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs
         const float* v0 = a.v + first * a.v_stride + (size_t)h * a.V + pb * COLS;
         const int chunks = max(1, v_cols / 4);
         auto copy = [&](int s) {
-            const int c0 = s * TPS, nt = min(TPS, n_new - c0), buf = s % STAGES;
+            const int c0 = s * TPS, nt = min(TPS, n_new - c0), buf = s % Plan::RING;
             if (lane == 0) {
                 // (in steps of single tokens the front of the one record is all that is wanted)
                 const int n = DELTA ? (nt + C - 1) / C * REC : nt * REC;
@@ -110,50 +117,53 @@ __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs
         // columns behind v's are zero in every stage; a last group that is not full is filled up with tokens that change
         // nothing and read nothing (the delta rule's records bring them)
         for (int i = v_cols + lane; i < COLS; i += 32)
-            for (int tt = 0; tt < STAGES * TPS; ++tt) vs[tt * COLS + i] = 0.f;
+            for (int tt = 0; tt < Plan::RING * TPS; ++tt) vs[tt * COLS + i] = 0.f;
         auto fill_up = [&](int s) {
-            const int nt = min(TPS, n_new - s * TPS), buf = s % STAGES;
+            const int nt = min(TPS, n_new - s * TPS), buf = s % Plan::RING;
             for (int tt = nt; tt < (nt + C - 1) / C * C; ++tt) {
                 for (int i = lane; i < COLS; i += 32) vs[(buf * TPS + tt) * COLS + i] = 0.f;
                 if (!DELTA)
                     for (int i = lane; i < 3 * Kp; i += 32) sm[buf * Plan::STAGE + tt * REC + i] = i < Kp ? 1.f : 0.f;
             }
         };
-        copy(0);
-        copies_commit();
-        if (n_stages > 1) copy(1);
-        copies_commit();
-        fill_up(0);
+        constexpr int AHEAD = Plan::RING - 1;
+#pragma unroll 1
+        for (int s = 0; s < max(1, AHEAD); ++s) {
+            if (s < n_stages) copy(s), fill_up(s);
+            copies_commit();
+        }
         bool ok = true;
         for (int s = 0; s < n_stages; ++s) {
-            copies_wait_all_but_one();               // stage s's values have landed, and so has
-            if (ok && !__all_sync(0xffffffffu, tc::mbar_wait(&full[s % STAGES], (uint32_t)(s / STAGES) & 1u, &never))) {
+            copies_wait<AHEAD == 0 ? 0 : AHEAD - 1>();           // stage s's values have landed, and so has
+            if (ok && !__all_sync(0xffffffffu, tc::mbar_wait(&full[s % Plan::RING], (uint32_t)(s / Plan::RING) & 1u, &never))) {
                 ok = false;                          // (its record never came: raise the flag and go on without waiting)
                 if (lane == 0) atomicExch(a.err, 9);
             }
             __syncthreads();                         // ... for everyone, and everyone is done with the stage before
-            if (s + 2 < n_stages) copy(s + 2);
+            if (AHEAD > 0 && s + AHEAD < n_stages) copy(s + AHEAD), fill_up(s + AHEAD);
             copies_commit();
-            if (s + 2 == n_stages) fill_up(s + 1);
         }
         if (!ok)                                     // what is still in flight lands before the block's memory goes away
-            for (int s = max(0, n_stages - STAGES); s < n_stages; ++s) tc::mbar_wait(&full[s % STAGES], (uint32_t)(s / STAGES) & 1u, &never);
+            for (int s = max(0, n_stages - Plan::RING); s < n_stages; ++s) tc::mbar_wait(&full[s % Plan::RING], (uint32_t)(s / Plan::RING) & 1u, &never);
         return;
     }
 
     const int l = tid % LG, col = tid / LG * CPT, c = pb * COLS + col;
+    // The lanes are shared out among the columns: a lane solves (delta rule) and writes the results of column `mine`.  It keeps
+    // column p ^ mine in place p, so that what it keeps in an exchange comes first.
+    const int mine = l / SHARE, in_share = l % SHARE;
     // pair 2 n + r of S: rows (n LG + l) 4 + 2 r and the one behind it
     f2 S[CPT][NP];
 #pragma unroll
     for (int p = 0; p < CPT; ++p)
 #pragma unroll
         for (int n = 0; n < N4; ++n) {
-            const int row = (n * LG + l) * 4;
-            const float* s = S_head + (size_t)(c + p) * a.K + row;
+            const int row = (n * LG + l) * 4, cc = c + (p ^ mine);
+            const float* s = S_head + (size_t)cc * a.K + row;
             float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (c + p < a.V && a.wide_state) {
+            if (cc < a.V && a.wide_state) {
                 if (row < a.K) f = *reinterpret_cast<const float4*>(s);
-            } else if (c + p < a.V) {
+            } else if (cc < a.V) {
                 if (row < a.K) f.x = s[0];
                 if (row + 1 < a.K) f.y = s[1];
                 if (row + 2 < a.K) f.z = s[2];
@@ -163,63 +173,96 @@ __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs
             S[p][2 * n + 1] = f2_of(f.z, f.w);
         }
     pdl_wait();
-    // the lanes are shared out among the columns: each solves (delta rule) and writes the results of its own
-    const int mine = CPT > 1 ? l / SHARE : 0, c_mine = c + mine;
-    float* yr = a.y + (size_t)first * a.H * a.V + (size_t)h * a.V + c_mine;
+    const int c_mine = c + mine;
     const size_t y_step = (size_t)a.H * a.V;
-    const bool writes = l % SHARE == 0 && c_mine < a.V;
+    float* yr = a.y + (size_t)first * y_step + (size_t)h * a.V + c_mine;
+    // the sums of N values per column over the lanes: column by column to its lanes, then value by value within them
+    auto reduce = [&](auto& dots, auto count) {
+        constexpr int N = decltype(count)::value;
+#pragma unroll
+        for (int w = CPT / 2, x = LG / 2; w >= 1; w /= 2, x /= 2)
+#pragma unroll
+            for (int n = 0; n < w * N; ++n) dots[n] += __shfl_xor_sync(0xffffffffu, dots[n + w * N], x);
+        scatter_sum<N, SHARE>(dots, lane);
+    };
+    int turn = 0;
     for (int s = 0; s < n_stages; ++s) {
         __syncthreads();
-        const int buf = s % STAGES, nt = min(TPS, n_new - s * TPS);
+        const int buf = s % Plan::RING, nt = min(TPS, n_new - s * TPS);
         const float* vb = vs + buf * TPS * COLS + col;
         for (int t0 = 0; t0 < nt; t0 += C) {
             const float* group = sm + buf * Plan::STAGE + (DELTA ? t0 / C : t0) * REC;
+            const ulonglong2* tok = reinterpret_cast<const ulonglong2*>(DELTA ? group + Kp + TABLE : group) + l;
             if constexpr (DELTA) {
-                const ulonglong2* tok = reinterpret_cast<const ulonglong2*>(group + Kp + TABLE) + l;         // 3 Kp / 4 a token
-                constexpr int ND = 2 * C * CPT;
-                float dots[ND];
+                float dots[2 * C * CPT];
 #pragma unroll
                 for (int j = 0; j < C; ++j) {
-                    f2 sk0[CPT], sk1[CPT], sq0[CPT], sq1[CPT];
+                    f2 sk[CPT], sq[CPT];
 #pragma unroll
                     for (int n = 0; n < N4; ++n) {
-                        const ulonglong2 fk = tok[j * (3 * Kp / 4) + n * LG], fq = tok[j * (3 * Kp / 4) + Kp / 4 + n * LG];
+                        const ulonglong2 fk = tok[j * V4 + n * LG], fq = tok[j * V4 + Kp / 4 + n * LG];
 #pragma unroll
                         for (int p = 0; p < CPT; ++p) {
-                            sk0[p] = n ? f2_fma(S[p][2 * n], fk.x, sk0[p]) : f2_mul(S[p][0], fk.x);
-                            sk1[p] = n ? f2_fma(S[p][2 * n + 1], fk.y, sk1[p]) : f2_mul(S[p][1], fk.y);
-                            sq0[p] = n ? f2_fma(S[p][2 * n], fq.x, sq0[p]) : f2_mul(S[p][0], fq.x);
-                            sq1[p] = n ? f2_fma(S[p][2 * n + 1], fq.y, sq1[p]) : f2_mul(S[p][1], fq.y);
+                            sk[p] = n ? f2_fma(S[p][2 * n], fk.x, sk[p]) : f2_mul(S[p][0], fk.x);
+                            sq[p] = n ? f2_fma(S[p][2 * n], fq.x, sq[p]) : f2_mul(S[p][0], fq.x);
+                            sk[p] = f2_fma(S[p][2 * n + 1], fk.y, sk[p]);
+                            sq[p] = f2_fma(S[p][2 * n + 1], fq.y, sq[p]);
                         }
                     }
 #pragma unroll
                     for (int p = 0; p < CPT; ++p) {
-                        dots[p * 2 * C + j] = f2_sum(f2_add(sk0[p], sk1[p]));
-                        dots[p * 2 * C + C + j] = f2_sum(f2_add(sq0[p], sq1[p]));
+                        dots[p * 2 * C + j] = f2_sum(sk[p]);
+                        dots[p * 2 * C + C + j] = f2_sum(sq[p]);
                     }
                 }
-                scatter_sum<ND, LG>(dots, lane);
-                using At = Scattered<ND, LG>;
-                constexpr int PER = At::per_lane, STR = At::stride;
+                reduce(dots, Int<2 * C>());
+                using At = Scattered<2 * C, SHARE>;
                 float all[2 * C];
 #pragma unroll
                 for (int i = 0; i < 2 * C; ++i)
-                    all[i] = __shfl_sync(0xffffffffu, dots[i % PER], mine * (2 * C / PER * STR) + i / PER * STR, LG);
+                    all[i] = SHARE == 1 ? dots[i] : __shfl_sync(0xffffffffu, dots[i % At::per_lane], i / At::per_lane * At::stride, SHARE);
                 const float4* gb = reinterpret_cast<const float4*>(group + Kp);
                 float u[C];
 #pragma unroll
                 for (int j = 0; j < C; ++j) {
-                    const float4 g = gb[j * 3], p0 = gb[j * 3 + 1], p1 = gb[j * 3 + 2];
-                    const float kk[3] = {p0.y, p0.w, p1.y}, kq[3] = {p0.z, p1.x, p1.z};
+                    const float4 p0 = gb[j * 2], p1 = j > 1 ? gb[j * 2 + 1] : make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float kk[3] = {p0.z, p1.x, p1.z}, kq[3] = {p0.w, p1.y, p1.w};
                     float b = all[j], o = all[C + j];
 #pragma unroll
                     for (int i = 0; i < j; ++i) {
                         b = fmaf(kk[(j - i - 1) % 3], u[i], b);
                         o = fmaf(kq[(j - i - 1) % 3], u[i], o);
                     }
-                    u[j] = g.y * (vb[(t0 + j) * COLS + mine] - b);
-                    o = fmaf(p0.x, u[j], o);
-                    if (writes && t0 + j < nt) yr[(s * TPS + t0 + j) * y_step] = o;
+                    u[j] = p0.x * (vb[(t0 + j) * COLS + mine] - b);
+                    o = fmaf(p0.y, u[j], o);
+                    if (in_share == 0 && c_mine < a.V && t0 + j < nt) yr[(s * TPS + t0 + j) * y_step] = o;
+                }
+                // every lane needs the u's of all its columns, as pairs
+                f2 uu[CPT][C];
+                if constexpr (CPT > 1 && C > 1) {
+                    f2* ub = us + (turn * COLS + col) * C;
+                    turn ^= 1;
+                    if (in_share == 0) {
+#pragma unroll
+                        for (int j = 0; j < C; j += 2)
+                            *reinterpret_cast<ulonglong2*>(ub + mine * C + j) = {f2_of(u[j], u[j]), f2_of(u[j + 1], u[j + 1])};
+                    }
+                    __syncwarp();
+#pragma unroll
+                    for (int p = 0; p < CPT; ++p)
+#pragma unroll
+                        for (int j = 0; j < C; j += 2) {
+                            const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(ub + (p ^ mine) * C + j);
+                            uu[p][j] = f.x, uu[p][j + 1] = f.y;
+                        }
+                } else {
+#pragma unroll
+                    for (int p = 0; p < CPT; ++p)
+#pragma unroll
+                        for (int j = 0; j < C; ++j) {
+                            const float up = CPT > 1 ? __shfl_sync(0xffffffffu, u[j], (p ^ mine) * SHARE, LG) : u[j];
+                            uu[p][j] = f2_of(up, up);
+                        }
                 }
                 const ulonglong2* gd = reinterpret_cast<const ulonglong2*>(group) + l;
 #pragma unroll
@@ -232,57 +275,47 @@ __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs
                     }
                 }
 #pragma unroll
-                for (int j = 0; j < C; ++j) {
-                    f2 uu[CPT];
-#pragma unroll
-                    for (int p = 0; p < CPT; ++p) {
-                        const float up = CPT > 1 ? __shfl_sync(0xffffffffu, u[j], p * SHARE, LG) : u[j];
-                        uu[p] = f2_of(up, up);
-                    }
+                for (int j = 0; j < C; ++j)
 #pragma unroll
                     for (int n = 0; n < N4; ++n) {
-                        const ulonglong2 fw = tok[j * (3 * Kp / 4) + 2 * (Kp / 4) + n * LG];
+                        const ulonglong2 fw = tok[j * V4 + 2 * (Kp / 4) + n * LG];
 #pragma unroll
                         for (int p = 0; p < CPT; ++p) {
-                            S[p][2 * n] = f2_fma(fw.x, uu[p], S[p][2 * n]);
-                            S[p][2 * n + 1] = f2_fma(fw.y, uu[p], S[p][2 * n + 1]);
+                            S[p][2 * n] = f2_fma(fw.x, uu[p][j], S[p][2 * n]);
+                            S[p][2 * n + 1] = f2_fma(fw.y, uu[p][j], S[p][2 * n + 1]);
                         }
                     }
-                }
             } else {
-                const ulonglong2* tok = reinterpret_cast<const ulonglong2*>(group) + l;
                 float dots[C * CPT];
 #pragma unroll
                 for (int j = 0; j < C; ++j) {
-                    f2 pp[CPT], sq0[CPT], sq1[CPT];
+                    f2 pp[CPT], sq[CPT];
 #pragma unroll
                     for (int p = 0; p < CPT; ++p) {
-                        const float pv = vb[(t0 + j) * COLS + p];
+                        const float pv = vb[(t0 + j) * COLS + (p ^ mine)];
                         pp[p] = f2_of(pv, pv);
                     }
 #pragma unroll
                     for (int n = 0; n < N4; ++n) {
-                        const ulonglong2 fd = tok[j * (3 * Kp / 4) + n * LG], fk = tok[j * (3 * Kp / 4) + Kp / 4 + n * LG];
-                        const ulonglong2 fq = tok[j * (3 * Kp / 4) + 2 * (Kp / 4) + n * LG];
+                        const ulonglong2 fd = tok[j * V4 + n * LG], fk = tok[j * V4 + Kp / 4 + n * LG], fq = tok[j * V4 + 2 * (Kp / 4) + n * LG];
 #pragma unroll
                         for (int p = 0; p < CPT; ++p) {
                             S[p][2 * n] = f2_fma(fk.x, pp[p], f2_mul(fd.x, S[p][2 * n]));
                             S[p][2 * n + 1] = f2_fma(fk.y, pp[p], f2_mul(fd.y, S[p][2 * n + 1]));
-                            sq0[p] = n ? f2_fma(S[p][2 * n], fq.x, sq0[p]) : f2_mul(S[p][0], fq.x);
-                            sq1[p] = n ? f2_fma(S[p][2 * n + 1], fq.y, sq1[p]) : f2_mul(S[p][1], fq.y);
+                            sq[p] = n ? f2_fma(S[p][2 * n], fq.x, sq[p]) : f2_mul(S[p][0], fq.x);
+                            sq[p] = f2_fma(S[p][2 * n + 1], fq.y, sq[p]);
                         }
                     }
 #pragma unroll
-                    for (int p = 0; p < CPT; ++p) dots[p * C + j] = f2_sum(f2_add(sq0[p], sq1[p]));
+                    for (int p = 0; p < CPT; ++p) dots[p * C + j] = f2_sum(sq[p]);
                 }
-                scatter_sum<C * CPT, LG>(dots, lane);
-                using At = Scattered<C * CPT, LG>;
-                if (l % At::stride == 0) {
+                reduce(dots, Int<C>());
+                using At = Scattered<C, SHARE>;
+                if (in_share % At::stride == 0 && c_mine < a.V) {
 #pragma unroll
                     for (int r = 0; r < At::per_lane; ++r) {
-                        const int i = l / At::stride * At::per_lane + r, p = i / C, j = t0 + i % C;
-                        if (p < CPT && j < nt && c + p < a.V)
-                            a.y[(size_t)(first + s * TPS + j) * y_step + (size_t)h * a.V + c + p] = dots[r] * a.q_scale;
+                        const int j = t0 + in_share / At::stride * At::per_lane + r;
+                        if (j < nt) yr[(s * TPS + j) * y_step] = dots[r] * a.q_scale;
                     }
                 }
             }
@@ -290,11 +323,12 @@ __global__ void __launch_bounds__(288) channel_scan_kernel(const ChannelScanArgs
     }
 #pragma unroll
     for (int p = 0; p < CPT; ++p) {
-        if (c + p >= a.V) break;
+        const int cc = c + (p ^ mine);
+        if (cc >= a.V) continue;
 #pragma unroll
         for (int n = 0; n < N4; ++n) {
             const int row = (n * LG + l) * 4;
-            float* s = S_head + (size_t)(c + p) * a.K + row;
+            float* s = S_head + (size_t)cc * a.K + row;
             float4 f;
             asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(S[p][2 * n]));
             asm("mov.b64 {%0, %1}, %2;" : "=f"(f.z), "=f"(f.w) : "l"(S[p][2 * n + 1]));

@@ -73,7 +73,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) channel_prepare_kernel(const 
         }
         if (lane < n_rec) {
             const float b = lane < nt ? sigmoid_f(a.proj[(size_t)(t + lane) * a.proj_stride + a.step_off + h]) : 0.f;
-            *reinterpret_cast<float4*>(ca.rec + ((size_t)h * ca.slots + slot) * delta_record(Kp) + Kp + lane * DELTA_ROW) = make_float4(1.f, b, 0.f, 0.f);
+            ca.rec[((size_t)h * ca.slots + slot) * delta_record(Kp) + Kp + lane * TOKEN_ROW] = b;
         }
         return;
     }
@@ -171,7 +171,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) channel_prepare_kernel(const 
         if (!(lane & 1)) {
             const int m = lane >> 1, c = m < 10 ? m - 4 : m - 10, back = c < 3 ? 1 : c < 5 ? 2 : 3;
             const int j = m < 4 ? m : (back == 1 ? c : back == 2 ? c - 3 : 0) + back;
-            if (j < n_rec) rec[Kp + j * DELTA_ROW + (m < 4 ? 4 : (m < 10 ? 3 : 4) + 2 * back)] = dots[0];
+            if (j < n_rec) rec[Kp + j * TOKEN_ROW + (m < 4 ? 1 : (m < 10 ? 0 : 1) + 2 * back)] = dots[0];
         }
     }
 }

@@ -6,17 +6,16 @@
 //   SIGMOID  out = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau), alone or as the first part of the records [decays | k | q] of a
 //            recurrence's scan (channel_memory.cuh), q and k copied from columns of the same rows
 //
-// The middle is a few dozen wide, so the result is bound by its own size; a block makes a tile of tokens by 64 columns,
-// both operands transposed in shared memory.  Sums run over r in ascending order, one fused multiply-add each, whatever the
-// tile, so a token's numbers do not depend on what else is in the step.  Two such products of the same step share a launch.
-#include "common.cuh"
+// A block makes a tile of tokens by 64 columns from rows of both operands in shared memory.  A sum runs over even and odd r side
+// by side, each in ascending order, whatever the tile, so a token's numbers do not depend on what else is in the step.  Two such products of the same step share a launch.
+#include "outer_memory.cuh"
 
 namespace {
 
+using namespace memory;
+
 enum : int { LR_PLAIN = 0, LR_DECAY = 1, LR_SIGMOID = 2 };
 constexpr int TN = 64, RC = 64, THREADS = 256;      // columns a block makes, how much of the middle is staged at a time
-
-__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 struct LowRankArgs {
     const float* a;
@@ -52,106 +51,113 @@ __device__ __forceinline__ void w_quad(const LowRankArgs& p, int n, int r, float
     for (int i = 0; i < 4; ++i) v[i] = r + i < p.R ? load_any(p.w, p.w_bf16 ? INFERO_BF16 : INFERO_F32, at + i) : 0.f;
 }
 
-// TM tokens: 64 (a thread makes 4 x 4 results) or 8 (2 x 1)
+// TM tokens: 64 (a thread makes 4 tokens by 4 columns, 16 apart) or 8 (2 x 1)
 template <int TM>
-__global__ void __launch_bounds__(THREADS) low_rank_kernel(const LowRankArgs first, const LowRankArgs second) {
-    constexpr int PT = TM == 64 ? 4 : 2, PN = TM == 64 ? 4 : 1;
-    __shared__ __align__(16) float as[RC][TM + 4], ws[RC][TN + 4];
+__global__ void __launch_bounds__(THREADS, 3) low_rank_kernel(const LowRankArgs first, const LowRankArgs second) {
+    constexpr bool BIG = TM == 64;
+    constexpr int PT = BIG ? 4 : 2, PN = BIG ? 4 : 1, STEP = 16;      // columns of a thread lie this far apart
+    __shared__ __align__(16) float as[TM][RC + 4], ws[TN][RC + 4];
+    float (*zs)[TN + 4] = reinterpret_cast<float (*)[TN + 4]>(&as[0][0]);       // the sums, in place of a's rows (RC = TN)
+    static_assert(RC == TN, "the sums take the place of a's rows");
     pdl_launch_dependents();
     LowRankArgs p = first;
     if (blockIdx.z) p = second;
     const int tid = threadIdx.x, n0 = blockIdx.x * TN, t0 = blockIdx.y * TM;
     if (n0 >= p.N) return;
-    const int tn = TM == 64 ? tid % 16 * 4 : tid % 64, tt = TM == 64 ? tid / 16 * 4 : tid / 64 * 2;
-    float acc[PT][PN], bias[PN], rate[PN];
+    const int tn = BIG ? tid % 16 : tid % 64, tt = BIG ? tid / 16 * 4 : tid / 64 * 2;
+    f2 acc[PT][PN];
 #pragma unroll
-    for (int j = 0; j < PN; ++j) {
-        const int n = n0 + tn + j;
-        bias[j] = p.bias && n < p.N ? p.bias[n] : 0.f;
-        rate[j] = p.mode == LR_DECAY && n < p.N ? -expf(p.a_log[n / p.per_head]) : -p.inv_tau;
+    for (int j = 0; j < PN; ++j)
 #pragma unroll
-        for (int i = 0; i < PT; ++i) acc[i][j] = 0.f;
-    }
-    // operands transposed: neighbouring threads take neighbouring rows, four numbers of each
+        for (int i = 0; i < PT; ++i) acc[i][j] = 0ull;
+    const int quad = tid % (RC / 4) * 4;             // a thread brings four neighbouring numbers of a row
     for (int r0 = 0; r0 < p.R; r0 += RC) {
-        const int nr = min(RC, p.R - r0);
         if (r0) __syncthreads();
-        for (int r = tid / TN * 4; r < nr; r += THREADS / TN * 4) {
+        constexpr int ROWS = THREADS / (RC / 4);     // rows of w a pass brings
+        float4 wv[TN / ROWS];
+#pragma unroll
+        for (int k = 0; k < TN / ROWS; ++k) {
+            const int n = tid / (RC / 4) + k * ROWS;
             float v[4] = {0.f, 0.f, 0.f, 0.f};
-            const int n = tid % TN;
-            if (n0 + n < p.N) w_quad(p, n0 + n, r0 + r, v);
-#pragma unroll
-            for (int i = 0; i < 4; ++i) ws[r + i][n] = v[i];
+            if (n0 + n < p.N && r0 + quad < p.R) w_quad(p, n0 + n, r0 + quad, v);
+            wv[k] = make_float4(v[0], v[1], v[2], v[3]);
         }
+#pragma unroll
+        for (int k = 0; k < TN / ROWS; ++k) *reinterpret_cast<float4*>(&ws[tid / (RC / 4) + k * ROWS][quad]) = wv[k];
         if (!r0) pdl_wait();                         // (the weights do not come from a kernel)
-        for (int r = tid / TM * 4; r < nr; r += THREADS / TM * 4) {
-            const int t = tid % TM;
-            const float* src = p.a + (t0 + t) * p.a_stride + r0 + r;
+        constexpr int PASS = THREADS / RC;           // rows of a a pass brings
+        const int ar = tid % RC, at = tid / RC;
+        const float* src = p.a + (t0 + at) * p.a_stride + r0 + ar;
+        float av[TM / PASS];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) as[r + i][t] = t0 + t < p.T && r + i < nr ? src[i] : 0.f;
-        }
+        for (int k = 0; k < TM / PASS; ++k) av[k] = t0 + at + k * PASS < p.T && r0 + ar < p.R ? src[k * PASS * p.a_stride] : 0.f;
+#pragma unroll
+        for (int k = 0; k < TM / PASS; ++k) as[at + k * PASS][ar] = av[k];
         __syncthreads();
-#pragma unroll 4
-        for (int r = 0; r < nr; ++r) {
-            float x[PT], y[PN];
-            if constexpr (TM == 64) {
-                const float4 f = *reinterpret_cast<const float4*>(&as[r][tt]), g = *reinterpret_cast<const float4*>(&ws[r][tn]);
-                x[0] = f.x, x[1] = f.y, x[2] = f.z, x[3] = f.w;
-                y[0] = g.x, y[1] = g.y, y[2] = g.z, y[3] = g.w;
-            } else {
-                x[0] = as[r][tt], x[1] = as[r][tt + 1], y[0] = ws[r][tn];
-            }
+        const int nr = min(RC, (p.R - r0 + 3) & ~3);
+#pragma unroll 2
+        for (int r = 0; r < nr; r += 4) {
+            ulonglong2 x[PT], y[PN];
+#pragma unroll
+            for (int i = 0; i < PT; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(&as[tt + i][r]);
+#pragma unroll
+            for (int j = 0; j < PN; ++j) y[j] = *reinterpret_cast<const ulonglong2*>(&ws[tn + j * STEP][r]);
 #pragma unroll
             for (int i = 0; i < PT; ++i)
 #pragma unroll
-                for (int j = 0; j < PN; ++j) acc[i][j] = fmaf(x[i], y[j], acc[i][j]);
+                for (int j = 0; j < PN; ++j) acc[i][j] = f2_fma(x[i].y, y[j].y, f2_fma(x[i].x, y[j].x, acc[i][j]));
         }
     }
-    const bool vec = PN == 4 && p.N % 4 == 0;
+    __syncthreads();
 #pragma unroll
-    for (int i = 0; i < PT; ++i) {
-        const int t = t0 + tt + i;
-        if (t >= p.T) break;
-        float* o = p.out + (size_t)t * p.N + n0 + tn;
-        float v[PN];
+    for (int i = 0; i < PT; ++i)
 #pragma unroll
-        for (int j = 0; j < PN; ++j) {
-            const float z = acc[i][j] + bias[j];
-            v[j] = p.mode == LR_PLAIN ? z : expf(rate[j] * softplus_f(p.mode == LR_DECAY ? z : -z));
+        for (int j = 0; j < PN; ++j) zs[tt + i][tn + j * STEP] = f2_sum(acc[i][j]);
+    __syncthreads();
+    // four neighbouring columns of a token at a time, always the same ones
+    const int c4 = tid % (TN / 4) * 4, n = n0 + c4, left = p.N - n;
+    if (left <= 0) return;
+    float bias[4], rate[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const int m = min(n + k, p.N - 1);
+        bias[k] = p.bias ? p.bias[m] : 0.f;
+        rate[k] = p.mode == LR_DECAY ? -expf(p.a_log[m / p.per_head]) : -p.inv_tau;
+    }
+    const int h = n / p.per_head, c = n - h * p.per_head;
+    const bool whole = left >= 4 && (p.N & 3) == 0 && (!p.rec || (((p.per_head | p.q_off | p.k_off | (int)p.qk_stride) & 3) == 0 &&
+                                                           (c + 4 < p.per_head || p.row_len == p.per_head)));
+#pragma unroll 1
+    for (int i = tid / (TN / 4); i < TM && t0 + i < p.T; i += THREADS / (TN / 4)) {
+        const int t = t0 + i;
+        const float4 f = *reinterpret_cast<const float4*>(&zs[i][c4]);
+        float v[4] = {f.x + bias[0], f.y + bias[1], f.z + bias[2], f.w + bias[3]};
+        if (p.mode != LR_PLAIN) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = expf(rate[k] * softplus_f(p.mode == LR_DECAY ? v[k] : -v[k]));
         }
-        if (p.rec) {
-            const float* row = p.qk + t * p.qk_stride;
-            if constexpr (PN == 4) {
-                const int n = n0 + tn, h = n / p.per_head, c = n - h * p.per_head;
-                if (n + 3 < p.N && ((p.per_head | p.q_off | p.k_off | (int)p.qk_stride) & 3) == 0 && c + 4 < p.per_head) {
-                    float* r = p.rec + ((size_t)h * p.T + t) * 3 * p.row_len + c;
-                    *reinterpret_cast<float4*>(r) = make_float4(v[0], v[1], v[2], v[3]);
-                    *reinterpret_cast<float4*>(r + p.row_len) = *reinterpret_cast<const float4*>(row + p.k_off + n);
-                    *reinterpret_cast<float4*>(r + 2 * p.row_len) = *reinterpret_cast<const float4*>(row + p.q_off + n);
-                    continue;
-                }
-            }
-#pragma unroll
-            for (int j = 0; j < PN; ++j) {
-                const int n = n0 + tn + j;
-                if (n >= p.N) break;
-                const int h = n / p.per_head, c = n - h * p.per_head;
-                float* r = p.rec + ((size_t)h * p.T + t) * 3 * p.row_len;
-                r[c] = v[j], r[p.row_len + c] = row[p.k_off + n], r[2 * p.row_len + c] = row[p.q_off + n];
-                if (c == p.per_head - 1)
-                    for (int i = p.per_head; i < p.row_len; ++i) r[i] = r[p.row_len + i] = r[2 * p.row_len + i] = 0.f;
-            }
+        if (!p.rec) {
+            float* o = p.out + (size_t)t * p.N + n;
+            if (whole) *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
+            else
+                for (int k = 0; k < min(4, left); ++k) o[k] = v[k];
             continue;
         }
-        if constexpr (PN == 4) {
-            if (vec && n0 + tn + 3 < p.N) {
-                *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
-                continue;
-            }
+        const float* row = p.qk + t * p.qk_stride;
+        if (whole) {
+            float* r = p.rec + ((size_t)h * p.T + t) * 3 * p.row_len + c;
+            *reinterpret_cast<float4*>(r) = make_float4(v[0], v[1], v[2], v[3]);
+            *reinterpret_cast<float4*>(r + p.row_len) = *reinterpret_cast<const float4*>(row + p.k_off + n);
+            *reinterpret_cast<float4*>(r + 2 * p.row_len) = *reinterpret_cast<const float4*>(row + p.q_off + n);
+            continue;
         }
-#pragma unroll
-        for (int j = 0; j < PN; ++j)
-            if (n0 + tn + j < p.N) o[j] = v[j];
+        for (int k = 0; k < min(4, left); ++k) {
+            const int hh = (n + k) / p.per_head, cc = n + k - hh * p.per_head;
+            float* r = p.rec + ((size_t)hh * p.T + t) * 3 * p.row_len;
+            r[cc] = v[k], r[p.row_len + cc] = row[p.k_off + n + k], r[2 * p.row_len + cc] = row[p.q_off + n + k];
+            if (cc == p.per_head - 1)
+                for (int m = p.per_head; m < p.row_len; ++m) r[m] = r[p.row_len + m] = r[2 * p.row_len + m] = 0.f;
+        }
     }
 }
 

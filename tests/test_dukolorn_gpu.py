@@ -297,6 +297,23 @@ def test_a_far_key_is_found_at_every_distance(dtype, back, D):
         assert _rel(PD.left_inner(h2.double(), w, "mix", m, EPS)[-1:], want[-1:]) > 0.05
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("H,G,D", [(4, 2, 64), (2, 1, 128), (6, 3, 48)])
+def test_single_tokens_behind_long_contexts(dtype, H, G, D):
+    """Contexts that the bf16 kernels cut into splits, beside a short one: sinks count once, however many splits there are."""
+    scale, cap, temp, n = D ** -0.5, 4.0, (0.3, 200), 1500
+    a = _left_alone(H, G, D, D, scale, 300, 16, cap, temp, dtype, gain=2.0, pages=128)
+    a.w["l0.mix.sink"] = a.w["l0.mix.sink"] + 6.0                          # (as much as a thousand keys)
+    _rebind(a)
+    m, w, d = left(H, G, D, D, scale, 300, cap, temp), a.weights(), a.spec.hidden
+    h1, h2 = _inputs(n, d, dtype, 1), _inputs(40, d, dtype, 2)
+    a.step([("a", h1[:n - 5]), ("b", h2[:35])])
+    got = [a.step([("a", h1[n - 5 + i:n - 4 + i]), ("b", h2[35 + i:36 + i])]) for i in range(5)]
+    tol = 3e-5 if dtype == "float32" else 3e-2
+    assert _rel(torch.cat([x["a"] for x in got])[:, :H * D], PD.left_inner(h1.double(), w, "mix", m, EPS)[-5:]) < tol
+    assert _rel(torch.cat([x["b"] for x in got])[:, :H * D], PD.left_inner(h2.double(), w, "mix", m, EPS)[-5:]) < tol
+
+
 def test_the_temperature_of_queries_far_out():
     """The factor at the positions where it steps, from the kernel that forms it: queries of unit norm times the factor."""
     from infero_b200.kernels import layer_ops as L
