@@ -289,7 +289,7 @@ def main(argv=None) -> int:
     ap.add_argument("--design-sizes", default="s,m")
     ap.add_argument("--design", default="vufizen", choices=["vufizen", "gositar", "banelix", "pibavik", "nuvarax", "dukolorn"],
                     help="with --designs: which of the added designs runs beside Qwen2 (pibavik: beside Banelix; nuvarax: beside Pibavik "
-                         "and Banelix, the closest designs)")
+                         "and Banelix; dukolorn: beside Nuvarax: the closest designs)")
     args = ap.parse_args(argv)
 
     if args.designs and args.impl != "reference":
